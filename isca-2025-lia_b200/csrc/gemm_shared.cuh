@@ -428,7 +428,7 @@ __device__ __forceinline__ void swap_epilogue_tile(const EpiParams& p, const Swa
   const bool two_shot = tp_on && (tp.opts & 128);    // fused all-reduce, world >= 4 (see the reduce side below)
   // two-shot: row group `it` (rows m0 + 8 it) of tile ta is reduced by rank (it + ta) % world.  Tracked incrementally as the
   // row groups are walked: a run-time modulo is ~30 dependent instructions, this code runs on one warp per scheduler with
-  // nothing to hide them behind, and one modulo per row group and destination cost ~5 us per exchange (ncu source view)
+  // nothing to hide them behind, and one modulo per row group and destination cost ~5 us per exchange
   int own_rank = two_shot ? w.ta % tp.world : 0;
   float* slot = ws + (size_t)cx.cta * (BN * TILE_A);
   constexpr int CH = BN >= 32 ? 32 : 16;
