@@ -32,7 +32,7 @@
 extern "C" {
 #endif
 
-#define LIA_ABI_VERSION 9
+#define LIA_ABI_VERSION 10
 
 typedef void* lia_stream_t; /* cudaStream_t */
 
@@ -483,6 +483,42 @@ int lia_diff_combine(const float* a, void* out, int act_f32, int M, int H, int G
 int lia_latent_prep_pairs(const void* q, int ldq, const void* dkv, int ldd, int act_f32, const float* c_norm_w, const double* freq, float mag,
                           const int* meta, void* cache, long long slot_stride, float* qa, int M, int H, int dim, int rot, int rot_dims,
                           int kv_rank, float eps, lia_stream_t stream);
+
+/* ---- Designs with a bigram embedding, wave positions, a latent cache without a rotated part under a sliding window with a sink,
+ * routers with sigmoid scores that weigh an expert's input, a gated shared expert.  (ABI 10) ---- */
+
+/* x[row] = table[id] + bigram[(prev * mul_prev + id * mul_cur) mod buckets] + wave in fp32; prev = the token before in the row's
+ * sequence, the bigram table has buckets + 1 rows and a sequence's first token takes the last one; tokens [slot][token_stride] int32
+ * holds the ids of every sequence so far (row meta[row] = {slot, position} writes its own); wave[2i] = sin(position * freq[i]),
+ * wave[2i+1] = cos of the same (freq: (W + 1) / 2 doubles).  bigram and freq may each be NULL.  The tables share a type.
+ * h (may be NULL) = w * x / sqrt(mean(x^2) + eps) in the given type. */
+int lia_embed_bigram_pos(const int64_t* ids, const void* table, const void* bigram, int table_f32, long long buckets, long long mul_prev,
+                         long long mul_cur, int* tokens, long long token_stride, const double* freq, const int* meta, float* x, const float* w,
+                         void* h, int h_f32, int rows, int W, int vocab, float eps, lia_stream_t stream);
+/* cache[slot][position] = c_norm_w * d / sqrt(mean(d^2) + eps), d = dkv[row][0..kv_rank): a latent cache row without a rotated part */
+int lia_latent_store(const void* dkv, int ldd, int act_f32, const float* c_norm_w, const int* meta, void* cache, long long slot_stride, int M,
+                     int kv_rank, float eps, lia_stream_t stream);
+/* lia_latent_attn with: window > 0 -- a query at position p attends to keys [p - window + 1, p] only (<= 0: its whole history);
+ * sink [H] (may be NULL) -- exp(sink[h]) joins the softmax's denominator as a term without key or value; rot may be 0 */
+int lia_latent_attn_masked(const float* qa, const void* cache, int cache_f32, long long slot_stride, const int* meta, const float* gate,
+                           const float* sink, float* out, float* workspace, int nsplit, int M, int H, int kv_rank, int rot, int window, float scale,
+                           lia_stream_t stream);
+/* lia_router_topk_ext on rows of ldl numbers whose first E are the logits; sigmoid != 0: an expert's score is the sigmoid of its logit */
+int lia_router_topk_scored(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int* idx, float* wt, int M, int E,
+                           int top, lia_stream_t stream);
+/* lia_gated_act on experts' projections in a plan's order: both factors of row m are first multiplied by wt[perm[m]] (0 where
+ * perm[m] < 0).  perm and wt NULL: lia_gated_act. */
+int lia_gated_act_weighted(const void* in, int ld, int up_off, void* out, int act_f32, int M, int F, int act, const int* perm, const float* wt,
+                           lia_stream_t stream);
+/* lia_moe_gemm_act with the routing weight on the experts' input (weigh_in != 0): up C = act of wt times the sums, down C = the sum */
+int lia_moe_gemm_weighted(const void* A, int a_f32, int lda, const void* W, int w_f32, long long w_expert_stride, void* C, int c_f32, int ldc,
+                          const int* perm, const int* tile_expert, int n_tiles, const int* idx, const float* wt, int pairs, int top, int N, int K,
+                          int up, int act, int gated, int n_real, float act_p0, float act_p1, int weigh_in, lia_stream_t stream);
+/* lia_moe_combine_ext with: weighted != 0 -- the experts' outputs carry their weights already (pos_of without wt); shared_gate
+ * (fp32, stride ldg, may be NULL) -- the shared expert's output times sigmoid(shared_gate[m * ldg]) */
+int lia_moe_combine_gated(const void* ypair, int ypair_f32, const int* pos_of, const float* wt, int weighted, const void* shared, int act_f32,
+                          const float* shared_gate, int ldg, const int* idx, int n_real, const void* h, float* y, int M, int W, int top,
+                          lia_stream_t stream);
 
 #ifdef __cplusplus
 }

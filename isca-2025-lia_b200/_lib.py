@@ -12,7 +12,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libliab200.so")
 
 EPI_BIAS, EPI_BIAS_RELU, EPI_BIAS_RESIDUAL, EPI_QKV = 0, 1, 2, 3
-ABI_VERSION = 9
+ABI_VERSION = 10
 TP_MAX_WORLD = 8
 P2P_HANDLE_BYTES = 64
 
@@ -166,6 +166,19 @@ _PROTOTYPES = {
     "lia_diff_combine": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p]),
     "lia_latent_prep_pairs": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_longlong, c_void_p,
                                       c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]),
+    # bigram embedding with wave positions, a latent cache without a rotated part under a window with a sink, sigmoid routers that
+    # weigh an expert's input, a gated shared expert
+    "lia_embed_bigram_pos": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p,
+                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]),
+    "lia_latent_store": (c_int, [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_float, c_void_p]),
+    "lia_latent_attn_masked": (c_int, [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                       c_int, c_int, c_int, c_float, c_void_p]),
+    "lia_router_topk_scored": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "lia_gated_act_weighted": (c_int, [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
+    "lia_moe_gemm_weighted": (c_int, [c_void_p, c_int, c_int, c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
+                                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "lia_moe_combine_gated": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p,
+                                      c_void_p, c_int, c_int, c_int, c_void_p]),
 }
 
 EXPORTS = tuple(_PROTOTYPES)

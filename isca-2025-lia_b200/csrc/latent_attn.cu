@@ -11,9 +11,12 @@
 //                 the same rotation of each head's rotated query part, written behind that head's q~ slot.
 //                 latent_prep_pairs is the same step with the rotation of neighbouring channels (2i, 2i+1) by angles from a
 //                 float64 frequency table (so that interpolated frequencies come from the host) and an amplitude on cos and sin.
+//   latent_store: the same RMS-norm for designs without a rotated part: the normalised latent alone becomes the cache row.
 //   latent_attn:  one block per (token, group of up to 8 heads, range of keys); 32 cached rows at a time are staged in shared
 //                 memory as fp32, scored (warp = head, lane = key), folded into a running softmax, and accumulated.  Few rows
-//                 and a long history (decoding): the keys are split over several blocks and a second kernel combines.
+//                 and a long history (decoding): the keys are split over several blocks and a second kernel combines.  A row
+//                 sees its whole history or the last `window` positions of it; a sink adds exp(sink[h]) to the softmax's
+//                 denominator, a term without key or value.
 #include <math.h>
 
 #include "common.cuh"
@@ -119,6 +122,23 @@ __global__ void __launch_bounds__(128) latent_prep_pairs_kernel(const T* __restr
   }
 }
 
+// cache[slot][pos] = cw * d / sqrt(mean(d^2) + eps) over the row's kv_rank numbers; one warp per token row
+template <typename T>
+__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ dkv, int ldd, const float* __restrict__ cw, const int* __restrict__ meta,
+                                                           T* __restrict__ cache, long long slot_stride, int M, int kv_rank, float eps) {
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= M) return;
+  const T* d = dkv + (size_t)row * ldd;
+  T* crow = cache + (size_t)meta[2 * row] * slot_stride + (size_t)meta[2 * row + 1] * kv_rank;
+  float ss = 0.f;
+  for (int i = lane; i < kv_rank; i += 32) {
+    const float v = ldf(d + i);
+    ss += v * v;
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)kv_rank + eps);
+  for (int i = lane; i < kv_rank; i += 32) stf(crow + i, ldf(d + i) * inv * cw[i]);
+}
+
 constexpr int TK = 32;     // cached rows per stage (= one warp's lanes: lane j scores key j)
 constexpr int HG = 8;      // heads per block (= warps per block: warp w scores head w)
 
@@ -133,14 +153,22 @@ __device__ __forceinline__ void load_vec(const float* p, float* f) {
 template <typename T> struct Vec { static constexpr int N = 8; };
 template <> struct Vec<float> { static constexpr int N = 4; };
 
+// 1 / the softmax's denominator for sums taken relative to the maximum m; a sink joins with exp(sink - m), and where it is the
+// larger one everything is taken relative to the sink instead (exp(sink - m) may overflow)
+__device__ __forceinline__ float over_denominator(float m, float l, const float* sink) {
+  if (sink == nullptr) return 1.0f / l;
+  const float top = fmaxf(m, *sink), a = expf(m - top);
+  return a / (l * a + expf(*sink - top));
+}
+
 // qa [M][H][D] fp32, cache [slot][capacity][D], out [M][H][kv_rank] fp32, times gate[M][H] (a per-head output gate) if
-// given.  RM = ceil(kv_rank / 256).  gridDim.z = nsplit: block z takes the z-th part of the row's keys; with nsplit > 1 the
+// given.  A row at position pos sees the cached rows max(0, pos - window + 1) .. pos.  RM = ceil(kv_rank / 256).  gridDim.z = nsplit: block z takes the z-th part of the row's keys; with nsplit > 1 the
 // unnormalised sums go to `part` ([M][H][nsplit][kv_rank]) and (max, sum) to `part_ml`, and latent_combine_kernel finishes.
 template <typename T, int RM>
 __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restrict__ qa, const T* __restrict__ cache, long long slot_stride,
-                                                          const int* __restrict__ meta, const float* __restrict__ gate, float* __restrict__ out,
-                                                          float* __restrict__ part, float2* __restrict__ part_ml, int H, int kv_rank, int rot,
-                                                          float scale) {
+                                                          const int* __restrict__ meta, const float* __restrict__ gate,
+                                                          const float* __restrict__ sink, float* __restrict__ out, float* __restrict__ part,
+                                                          float2* __restrict__ part_ml, int H, int kv_rank, int rot, int window, float scale) {
   extern __shared__ __align__(16) float sm[];
   const int D = kv_rank + rot, DS = padded_row(D), G4 = (DS - 4) / 4;
   float* qs = sm;                    // [HG][DS]
@@ -155,8 +183,9 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
   const int slot = meta[2 * row], pos = meta[2 * row + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* crows = cache + (size_t)slot * slot_stride;
-  const int tiles = (pos + TK) / TK, per = (tiles + nsplit - 1) / nsplit;
-  const int j_begin = z * per * TK, j_end = min(pos + 1, (z + 1) * per * TK);
+  const int first = max(0, pos - window + 1);
+  const int tiles = (pos - first + TK) / TK, per = (tiles + nsplit - 1) / nsplit;
+  const int j_begin = first + z * per * TK, j_end = min(pos + 1, first + (z + 1) * per * TK);
   constexpr int VEC = Vec<T>::N;
   const bool vec = (D % VEC == 0) && (slot_stride % VEC == 0) && (reinterpret_cast<uintptr_t>(cache) % 16 == 0);
 
@@ -275,7 +304,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
     if (hh < nh) {
       const size_t rh = (size_t)row * H + h0 + hh;
       if (nsplit == 1) {
-        const float invl = (gate ? gate[rh] : 1.0f) / lsum[hh];
+        const float invl = (gate ? gate[rh] : 1.0f) * over_denominator(msum[hh], lsum[hh], sink ? sink + h0 + hh : nullptr);
 #pragma unroll
         for (int i = 0; i < RM; ++i) {
           const int r = threadIdx.x + 256 * i;
@@ -293,15 +322,17 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const float* __restric
   }
 }
 
-// out[rh] = gate * sum_z part[rh][z] e^(m_z - m) / sum_z l_z e^(m_z - m), m = max_z m_z (a part without keys has m = -inf, l = 0)
+// out[rh] = gate * sum_z part[rh][z] e^(m_z - m) / (sum_z l_z e^(m_z - m) + e^(sink - m)), m = max_z m_z (a part without keys has
+// m = -inf, l = 0)
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part, const float2* __restrict__ part_ml,
-                                                             const float* __restrict__ gate, float* __restrict__ out, int kv_rank, int nsplit) {
+                                                             const float* __restrict__ gate, const float* __restrict__ sink, float* __restrict__ out,
+                                                             int H, int kv_rank, int nsplit) {
   const size_t rh = blockIdx.x;
   float m = -INFINITY;
   for (int z = 0; z < nsplit; ++z) m = fmaxf(m, part_ml[rh * nsplit + z].x);
   float l = 0.f;
   for (int z = 0; z < nsplit; ++z) l += part_ml[rh * nsplit + z].y * expf(part_ml[rh * nsplit + z].x - m);
-  const float g = (gate ? gate[rh] : 1.0f) / l;
+  const float g = (gate ? gate[rh] : 1.0f) * over_denominator(m, l, sink ? sink + rh % H : nullptr);
   for (int r = threadIdx.x; r < kv_rank; r += 128) {
     float s = 0.f;
     for (int z = 0; z < nsplit; ++z) s = fmaf(part[(rh * nsplit + z) * kv_rank + r], expf(part_ml[rh * nsplit + z].x - m), s);
@@ -310,8 +341,8 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
 }
 
 template <typename T, int RM>
-int launch_attn(const float* qa, const void* cache, long long slot_stride, const int* meta, const float* gate, float* out, float* ws, int nsplit,
-                int M, int H, int kv_rank, int rot, float scale, cudaStream_t stream) {
+int launch_attn(const float* qa, const void* cache, long long slot_stride, const int* meta, const float* gate, const float* sink, float* out, float* ws,
+                int nsplit, int M, int H, int kv_rank, int rot, int window, float scale, cudaStream_t stream) {
   const int DS = padded_row(kv_rank + rot);
   const size_t smem = ((size_t)HG * DS + (size_t)TK * DS + HG * TK + 3 * HG + 8 * HG * TK) * sizeof(float);
   LIA_CHECK_ARG(smem <= 200 * 1024, "lia_latent_attn: a cache row of %d numbers does not fit the shared-memory stage", kv_rank + rot);
@@ -319,22 +350,22 @@ int launch_attn(const float* qa, const void* cache, long long slot_stride, const
   dim3 grid(M, (H + HG - 1) / HG, nsplit);
   float* part = ws;
   float2* part_ml = reinterpret_cast<float2*>(ws + (size_t)M * H * nsplit * kv_rank);
-  latent_attn_kernel<T, RM><<<grid, 256, smem, stream>>>(qa, reinterpret_cast<const T*>(cache), slot_stride, meta, gate, out, part, part_ml, H,
-                                                         kv_rank, rot, scale);
+  latent_attn_kernel<T, RM><<<grid, 256, smem, stream>>>(qa, reinterpret_cast<const T*>(cache), slot_stride, meta, gate, sink, out, part, part_ml,
+                                                         H, kv_rank, rot, window, scale);
   LIA_LAUNCH_CHECK();
   if (nsplit > 1) {
-    latent_combine_kernel<<<(unsigned)((size_t)M * H), 128, 0, stream>>>(part, part_ml, gate, out, kv_rank, nsplit);
+    latent_combine_kernel<<<(unsigned)((size_t)M * H), 128, 0, stream>>>(part, part_ml, gate, sink, out, H, kv_rank, nsplit);
     LIA_LAUNCH_CHECK();
   }
   return LIA_OK;
 }
 
 template <typename T>
-int dispatch_attn(const float* qa, const void* cache, long long slot_stride, const int* meta, const float* gate, float* out, float* ws, int nsplit,
-                  int M, int H, int kv_rank, int rot, float scale, cudaStream_t stream) {
-  if (kv_rank <= 256) return launch_attn<T, 1>(qa, cache, slot_stride, meta, gate, out, ws, nsplit, M, H, kv_rank, rot, scale, stream);
-  if (kv_rank <= 512) return launch_attn<T, 2>(qa, cache, slot_stride, meta, gate, out, ws, nsplit, M, H, kv_rank, rot, scale, stream);
-  return launch_attn<T, 4>(qa, cache, slot_stride, meta, gate, out, ws, nsplit, M, H, kv_rank, rot, scale, stream);
+int dispatch_attn(const float* qa, const void* cache, long long slot_stride, const int* meta, const float* gate, const float* sink, float* out, float* ws,
+                  int nsplit, int M, int H, int kv_rank, int rot, int window, float scale, cudaStream_t stream) {
+  if (kv_rank <= 256) return launch_attn<T, 1>(qa, cache, slot_stride, meta, gate, sink, out, ws, nsplit, M, H, kv_rank, rot, window, scale, stream);
+  if (kv_rank <= 512) return launch_attn<T, 2>(qa, cache, slot_stride, meta, gate, sink, out, ws, nsplit, M, H, kv_rank, rot, window, scale, stream);
+  return launch_attn<T, 4>(qa, cache, slot_stride, meta, gate, sink, out, ws, nsplit, M, H, kv_rank, rot, window, scale, stream);
 }
 
 }  // namespace
@@ -382,10 +413,33 @@ extern "C" size_t lia_latent_attn_workspace_floats(int M, int H, int kv_rank, in
 
 extern "C" int lia_latent_attn(const float* qa, const void* cache, int cache_f32, long long slot_stride, const int* meta, const float* gate,
                                float* out, float* workspace, int nsplit, int M, int H, int kv_rank, int rot, float scale, lia_stream_t stream_) {
+  return lia_latent_attn_masked(qa, cache, cache_f32, slot_stride, meta, gate, nullptr, out, workspace, nsplit, M, H, kv_rank, rot, 0, scale, stream_);
+}
+
+// window > 0: the last `window` positions only (<= 0: the whole history); sink [H] (may be null): a further term of the denominator
+extern "C" int lia_latent_attn_masked(const float* qa, const void* cache, int cache_f32, long long slot_stride, const int* meta, const float* gate,
+                                      const float* sink, float* out, float* workspace, int nsplit, int M, int H, int kv_rank, int rot, int window,
+                                      float scale, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(qa && cache && meta && out, "lia_latent_attn: null pointer");
   LIA_CHECK_ARG(M > 0 && H > 0 && H <= 65535 * HG && kv_rank > 0 && kv_rank <= 1024 && rot >= 0, "lia_latent_attn: bad shape M=%d H=%d kv_rank=%d rot=%d", M, H, kv_rank, rot);
   LIA_CHECK_ARG(nsplit >= 1 && nsplit <= 64 && (nsplit == 1 || workspace != nullptr), "lia_latent_attn: %d key ranges need a workspace", nsplit);
-  if (cache_f32) return dispatch_attn<float>(qa, cache, slot_stride, meta, gate, out, workspace, nsplit, M, H, kv_rank, rot, scale, stream);
-  return dispatch_attn<bf16>(qa, cache, slot_stride, meta, gate, out, workspace, nsplit, M, H, kv_rank, rot, scale, stream);
+  if (window <= 0) window = 1 << 30;
+  if (cache_f32) return dispatch_attn<float>(qa, cache, slot_stride, meta, gate, sink, out, workspace, nsplit, M, H, kv_rank, rot, window, scale, stream);
+  return dispatch_attn<bf16>(qa, cache, slot_stride, meta, gate, sink, out, workspace, nsplit, M, H, kv_rank, rot, window, scale, stream);
+}
+
+extern "C" int lia_latent_store(const void* dkv, int ldd, int act_f32, const float* c_norm_w, const int* meta, void* cache, long long slot_stride,
+                                int M, int kv_rank, float eps, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(dkv && c_norm_w && meta && cache && M > 0 && kv_rank > 0 && ldd >= kv_rank, "lia_latent_store: bad arguments");
+  const unsigned grid = (unsigned)((M + 3) / 4);
+  if (act_f32)
+    latent_store_kernel<float><<<grid, 128, 0, stream>>>(reinterpret_cast<const float*>(dkv), ldd, c_norm_w, meta, reinterpret_cast<float*>(cache),
+                                                         slot_stride, M, kv_rank, eps);
+  else
+    latent_store_kernel<bf16><<<grid, 128, 0, stream>>>(reinterpret_cast<const bf16*>(dkv), ldd, c_norm_w, meta, reinterpret_cast<bf16*>(cache),
+                                                        slot_stride, M, kv_rank, eps);
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
 }

@@ -1,6 +1,6 @@
 // Row operations of models that keep their residual stream in 32-bit floats: RMS norms with a scalar or a per-channel
 // weight (fused with the residual add that follows a sublayer and with the norm that precedes the next one), the token
-// embedding with its norm, the gated, normed residual update with a weighted mix of all earlier layers' results, the
+// embedding with its norm, with learned or wave positions and with a bigram table, the gated, normed residual update with a weighted mix of all earlier layers' results, the
 // polynomial activation between norms, a gated feed-forward activation with clamps, a projection onto a handful of outputs with the
 // gate non-linearities in its epilogue, a plain strided-batched projection on the CUDA cores (true 32-bit products and
 // sums: the exact path, and the carrier of shapes the tensor-core GEMM does not take), and a 32-bit argmax.
@@ -109,6 +109,56 @@ __global__ void __launch_bounds__(256) embed_scale_pos_kernel(const int64_t* __r
       stf(cat + (size_t)row * 2 * W + W + i, v);
     }
   }
+}
+
+// Designs whose embedding also looks at the token before, and whose positions are sine and cosine waves:
+//   x[row] = table[id] + bigram[(prev * mul_prev + id * mul_cur) mod buckets] + wave(position)
+// A sequence's first token takes the bigram table's last row (number `buckets`).  The token before a portion's first row comes
+// from tokens [slot][capacity], the ids of the sequence so far; every row leaves its own id there.  wave(p)[2i] = sin(p * freq[i]),
+// wave(p)[2i+1] = cos of the same: the angle is a float64 product brought into [-pi, pi] before it is rounded to fp32.
+//   h (may be null): the norm that the first layer reads, w * x / sqrt(mean(x^2) + eps).
+// `bigram` and `freq` may each be null.  `xs` (dynamic shared memory, W floats) keeps the row for the norm.
+template <typename T, typename TH>
+__global__ void __launch_bounds__(256) embed_bigram_pos_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, const T* __restrict__ bigram,
+                                                               long long buckets, long long mul_prev, long long mul_cur, int* __restrict__ tokens,
+                                                               long long token_stride, const double* __restrict__ freq, const int* __restrict__ meta,
+                                                               float* __restrict__ x, const float* __restrict__ w, TH* __restrict__ h, int W, int vocab,
+                                                               float eps) {
+  extern __shared__ float xs[];
+  __shared__ float red[8];
+  const int row = blockIdx.x, slot = meta[2 * row], p = meta[2 * row + 1];
+  long long id = ids[row];
+  if (id < 0 || id >= vocab) id = 0;     // the host checks the range; never read outside the table
+  const T* e = table + (size_t)id * W;
+  const T* b = nullptr;
+  if (bigram != nullptr) {
+    long long at = buckets;
+    if (p > 0) {
+      const bool inside = row > 0 && meta[2 * (row - 1)] == slot && meta[2 * (row - 1) + 1] == p - 1;     // rows of a portion follow each other
+      const long long prev = inside ? ids[row - 1] : (long long)tokens[(size_t)slot * token_stride + p - 1];
+      at = (prev * mul_prev + id * mul_cur) % buckets;
+      if (at < 0) at += buckets;
+    }
+    b = bigram + (size_t)at * W;
+    if (threadIdx.x == 0) tokens[(size_t)slot * token_stride + p] = (int)id;
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    float v = ldf(e + i);
+    if (b != nullptr) v += ldf(b + i);
+    if (freq != nullptr) {
+      const double a = (double)p * freq[i >> 1];
+      const float r = (float)(a - rint(a * 0.15915494309189533577) * 6.28318530717958647693);
+      v += (i & 1) ? cosf(r) : sinf(r);
+    }
+    x[(size_t)row * W + i] = v;
+    xs[i] = v;
+    ss += v * v;
+  }
+  if (h == nullptr) return;
+  ss = block_sum<256>(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)W + eps);
+  for (int i = threadIdx.x; i < W; i += 256) stf(h + (size_t)row * W + i, xs[i] * inv * w[i]);
 }
 
 // The residual update of pre-norm designs, fused with the norm (or the plain cast) that the next sublayer reads:
@@ -685,6 +735,30 @@ extern "C" int lia_softcap_f32(float* x, long long n, float cap, lia_stream_t st
   const size_t capb = (size_t)lia_sm_count() * 16;
   if (blocks > capb) blocks = capb;
   softcap_kernel<<<(unsigned)blocks, 256, 0, stream>>>(x, (size_t)n, cap);
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
+}
+
+extern "C" int lia_embed_bigram_pos(const int64_t* ids, const void* table, const void* bigram, int table_f32, long long buckets, long long mul_prev,
+                                    long long mul_cur, int* tokens, long long token_stride, const double* freq, const int* meta, float* x, const float* w,
+                                    void* h, int h_f32, int rows, int W, int vocab, float eps, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(ids && table && meta && x && rows > 0 && W > 0 && vocab > 0 && (size_t)W * 4 <= 160 * 1024, "lia_embed_bigram_pos: bad arguments");
+  LIA_CHECK_ARG(!bigram || (tokens && token_stride > 0 && buckets > 0), "lia_embed_bigram_pos: the bigram table needs its height and the sequences' ids");
+  LIA_CHECK_ARG(!h || w, "lia_embed_bigram_pos: the norm needs its weight");
+  const size_t smem = (size_t)W * sizeof(float);
+#define LIA_EBP(T, TH)                                                                                                       \
+  do {                                                                                                                       \
+    if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(embed_bigram_pos_kernel<T, TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    embed_bigram_pos_kernel<T, TH><<<rows, 256, smem, stream>>>(ids, reinterpret_cast<const T*>(table), reinterpret_cast<const T*>(bigram), buckets, \
+                                                                mul_prev, mul_cur, tokens, token_stride, freq, meta, x, w, reinterpret_cast<TH*>(h), \
+                                                                W, vocab, eps);                                              \
+  } while (0)
+  if (table_f32 && h_f32) LIA_EBP(float, float);
+  else if (table_f32) LIA_EBP(float, bf16);
+  else if (h_f32) LIA_EBP(bf16, float);
+  else LIA_EBP(bf16, bf16);
+#undef LIA_EBP
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }

@@ -4,12 +4,12 @@
 //   ln_add_norm    x += mult * LN_post(y);  x += extra;  h = LN_pre(x)    (each part optional, one pass over the row)
 //   ln_gather      h[r] = LN(x[rows[r]]) for the few rows whose logits are wanted
 //   gated_act      out = act(gate) * up  (or act(gate) alone) on column ranges of one projection's output
-//   router_topk    softmax over the experts' logits, the `top` largest (by score, or by score plus a correction), renormalised or not
+//   router_topk    softmax over the experts' logits or a sigmoid of each, the `top` largest (by score, or by score plus a correction), renormalised or not
 //   moe_plan       (token, choice) pairs grouped by expert into row tiles
 //   moe_gemm       one projection of every expert over its own rows (gather on the way in, activation or routing weight on
 //                  the way out); moe_fewrows does the same for a handful of pairs with one warp per output
 //   moe_gather     the experts' input rows laid out in the plan's order, for projections that want contiguous rows
-//   moe_combine    y[token] = sum over its choices (+ the shared expert's output); identity experts hand the token itself back
+//   moe_combine    y[token] = sum over its choices (+ the shared expert's output, behind a gate or not); identity experts hand the token itself back
 // LN is (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b with fp32 statistics taken in two passes over a staged row.
 #include <math.h>
 
@@ -131,44 +131,58 @@ __device__ __forceinline__ float gated_apply(float g, float u, int act, float p0
 }
 
 // out[m][f] = act(in[m][f]) * in[m][up_off + f]   (up_off < 0: no second factor)
+// perm (may be null): row m holds the projections of pair perm[m], whose routing weight multiplies both factors first (the
+// projection of a weighted input); rows of no pair (-1) become zero.
 template <typename T>
-__global__ void gated_act_kernel(const T* __restrict__ in, int ld, int up_off, T* __restrict__ out, int M, int F, int act) {
+__global__ void gated_act_kernel(const T* __restrict__ in, int ld, int up_off, T* __restrict__ out, int M, int F, int act,
+                                 const int* __restrict__ perm, const float* __restrict__ wt) {
   const size_t n = (size_t)M * F;
   for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
     const size_t m = e / F;
     const int f = (int)(e - m * F);
-    float v = act_apply(ldf(in + m * ld + f), act);
-    if (up_off >= 0) v *= ldf(in + m * ld + up_off + f);
+    float ws = 1.0f;
+    if (perm != nullptr) ws = perm[m] < 0 ? 0.f : wt[perm[m]];
+    float v = act_apply(ws * ldf(in + m * ld + f), act);
+    if (up_off >= 0) v *= ws * ldf(in + m * ld + up_off + f);
     stf(out + e, v);
   }
 }
 
 // ---------------------------------------------------------------------------------------------------- router
-// One warp per token: softmax over E logits (fp32), then `top` rounds of arg-max (lowest index on ties) over the scores
-// plus an optional per-expert correction that takes part in the choice only; a chosen expert's weight is its plain
-// score, divided by their sum (+ 1e-20) when `renorm` is set.
-__global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ idx,
-                                                          float* __restrict__ wt, int M, int E, int top, int renorm) {
+// One warp per token: softmax over E logits (fp32), or a sigmoid of each (`sigmoid`), then `top` rounds of arg-max (lowest
+// index on ties) over the scores plus an optional per-expert correction that takes part in the choice only; a chosen expert's
+// weight is its plain score, divided by their sum (+ 1e-20) when `renorm` is set.  Sigmoid scores without a correction are
+// compared by their logits (the same order, also where the scores round to 1).
+__global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ correction,
+                                                          int* __restrict__ idx, float* __restrict__ wt, int M, int E, int top, int renorm,
+                                                          int sigmoid) {
   extern __shared__ float sc[];          // [4 warps][2][E]: scores, choice scores
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row = blockIdx.x * 4 + warp;
   if (row >= M) return;
   float* s = sc + warp * 2 * E;
   float* ch = s + E;
-  const float* z = logits + (size_t)row * E;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float p = expf(z[e] - mx);
-    s[e] = p;
-    sum += p;
-  }
-  sum = warp_sum(sum);
-  for (int e = lane; e < E; e += 32) {
-    s[e] = s[e] / sum;
-    ch[e] = s[e] + (correction ? correction[e] : 0.f);
+  const float* z = logits + (size_t)row * ldl;
+  if (sigmoid) {
+    for (int e = lane; e < E; e += 32) {
+      s[e] = 1.0f / (1.0f + expf(-z[e]));
+      ch[e] = correction ? s[e] + correction[e] : z[e];
+    }
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(z[e] - mx);
+      s[e] = p;
+      sum += p;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      s[e] = s[e] / sum;
+      ch[e] = s[e] + (correction ? correction[e] : 0.f);
+    }
   }
   __syncwarp();
   float chosen_sum = 0.f;
@@ -241,10 +255,12 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
 // 64 x 64 tile, 16-wide k slabs, 4 x 4 outputs per thread, fp32 products and sums in k order (as the plain projection).
 // GATED (UP only): an expert's weights are [2N][K], N gate rows then N up rows, and C = act(gate sum) * (up sum).
 // Tiles of experts >= n_real (experts without weights, whose pairs the combining step serves) are skipped.
+// weigh_in: the routing weight multiplies the expert's input -- both UP sums before the activation -- and not the DOWN sum.
 template <typename TA, typename TW, typename TC, bool UP, bool GATED>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ Wt, long long sW, TC* __restrict__ C,
                                                        int ldc, const int* __restrict__ perm, const int* __restrict__ tile_expert,
-                                                       const float* __restrict__ wt, int top, int N, int K, int act, int n_real, float p0, float p1) {
+                                                       const float* __restrict__ wt, int top, int N, int K, int act, int n_real, float p0, float p1,
+                                                       int weigh_in) {
   const int e = tile_expert[blockIdx.y];
   if (e < 0 || e >= n_real) return;
   __shared__ float As[16][TM + 4];
@@ -302,12 +318,13 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
     const int r = ty * 4 + i;
     const int p = dstp[r];
     if (p < 0) continue;
+    const float ws = (UP ? weigh_in : !weigh_in) ? wt[p] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
-      if (UP) stf(C + (size_t)(row0 + r) * ldc + n, GATED ? gated_apply(acc[i][j], accu[i][j], act, p0, p1) : act_apply(acc[i][j], act));
-      else stf(C + (size_t)p * ldc + n, acc[i][j] * wt[p]);
+      if (UP) stf(C + (size_t)(row0 + r) * ldc + n, GATED ? gated_apply(ws * acc[i][j], ws * accu[GATED ? i : 0][j], act, p0, p1) : act_apply(ws * acc[i][j], act));
+      else stf(C + (size_t)p * ldc + n, acc[i][j] * ws);
     }
   }
 }
@@ -334,11 +351,11 @@ __device__ __forceinline__ void load8(const float* p, int k, int K, bool vec, fl
 // The same projections for a handful of pairs (decoding): one warp per output n of pair p reads row n of expert idx[p]
 // with 128-bit loads; memory-bound on the chosen experts' weights.  UP: A row = token p / top, C row = p, act applied.
 // DOWN: A row = p, C row = p, times wt[p].  gated (UP): row N + n of the expert is the second factor, C = act(gate) * up.
-// Pairs of experts >= n_real are skipped.
+// Pairs of experts >= n_real are skipped; weigh_in as in moe_gemm_kernel.
 template <typename TA, typename TW, typename TC, bool UP>
 __global__ void __launch_bounds__(128) moe_fewrows_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ Wt, long long sW, TC* __restrict__ C,
                                                           int ldc, const int* __restrict__ idx, const float* __restrict__ wt, int top, int N, int K,
-                                                          int act, int gated, int n_real, float p0, float p1) {
+                                                          int act, int gated, int n_real, float p0, float p1, int weigh_in) {
   const int p = blockIdx.y, n = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (n >= N || idx[p] >= n_real) return;
   const TW* wr = Wt + (size_t)idx[p] * sW + (size_t)n * K;
@@ -360,7 +377,10 @@ __global__ void __launch_bounds__(128) moe_fewrows_kernel(const TA* __restrict__
   }
   acc = warp_sum(acc);
   if (UP && gated) accu = warp_sum(accu);
-  if (lane == 0) stf(C + (size_t)p * ldc + n, UP ? (gated ? gated_apply(acc, accu, act, p0, p1) : act_apply(acc, act)) : acc * wt[p]);
+  if (lane == 0) {
+    const float ws = (UP ? weigh_in : !weigh_in) ? wt[p] : 1.0f;
+    stf(C + (size_t)p * ldc + n, UP ? (gated ? gated_apply(ws * acc, ws * accu, act, p0, p1) : act_apply(ws * acc, act)) : acc * ws);
+  }
 }
 
 // dst[place] = src[perm[place] / top] for every place of the plan, zeros in the padding: the experts' inputs, expert by expert
@@ -375,13 +395,14 @@ __global__ void moe_gather_kernel(const T* __restrict__ src, const int* __restri
   }
 }
 
-// y[m][c] = sum_t f(m * top + t)[c] (in the order of t) + shared[m][c];  f(pair) = ypair[pair], or, with a plan,
-// wt[pair] * ypair[pos_of[pair]] (the experts' outputs still in the plan's order and not yet weighted).  A pair whose expert
+// y[m][c] = sum_t f(m * top + t)[c] (in the order of t) + sigmoid(sgate[m]) * shared[m][c] (sgate null: + shared[m][c]);
+// f(pair) = ypair[pair], or, with a plan, wt[pair] * ypair[pos_of[pair]] (the experts' outputs still in the plan's order and not
+// yet weighted; `weighted`: nor to be).  A pair whose expert
 // idx[pair] >= n_real is an identity expert: f(pair) = wt[pair] * h[m], and ypair is not read for it.
 template <typename TY, typename TS>
 __global__ void moe_combine_kernel(const TY* __restrict__ ypair, const int* __restrict__ pos_of, const float* __restrict__ wt,
                                    const TS* __restrict__ shared, float* __restrict__ y, int M, int W, int top, const int* __restrict__ idx,
-                                   int n_real, const TS* __restrict__ h) {
+                                   int n_real, const TS* __restrict__ h, int weighted, const float* __restrict__ sgate, int ldg) {
   const size_t n = (size_t)M * W;
   for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
     const size_t m = e / W;
@@ -390,10 +411,10 @@ __global__ void moe_combine_kernel(const TY* __restrict__ ypair, const int* __re
     for (int t = 0; t < top; ++t) {
       const size_t pair = m * top + t;
       if (idx && idx[pair] >= n_real) s = fmaf(wt[pair], ldf(h + e), s);
-      else if (pos_of) s = fmaf(wt[pair], ldf(ypair + (size_t)pos_of[pair] * W + c), s);
+      else if (pos_of) s = fmaf(weighted ? 1.0f : wt[pair], ldf(ypair + (size_t)pos_of[pair] * W + c), s);
       else s += ldf(ypair + pair * W + c);
     }
-    if (shared) s += ldf(shared + e);
+    if (shared) s += sgate ? ldf(shared + e) / (1.0f + expf(-sgate[m * ldg])) : ldf(shared + e);
     y[e] = s;
   }
 }
@@ -456,12 +477,18 @@ extern "C" int lia_ln_gather(const float* x, const int* rows, const float* w, co
 }
 
 extern "C" int lia_gated_act(const void* in, int ld, int up_off, void* out, int act_f32, int M, int F, int act, lia_stream_t stream_) {
+  return lia_gated_act_weighted(in, ld, up_off, out, act_f32, M, F, act, nullptr, nullptr, stream_);
+}
+
+extern "C" int lia_gated_act_weighted(const void* in, int ld, int up_off, void* out, int act_f32, int M, int F, int act, const int* perm,
+                                      const float* wt, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(in && out && M > 0 && F > 0 && ld >= F && (up_off < 0 || (up_off >= F && ld >= up_off + F)), "lia_gated_act: bad arguments");
+  LIA_CHECK_ARG((perm == nullptr) == (wt == nullptr), "lia_gated_act: a row order and routing weights go together");
   LIA_CHECK_ARG(act >= LIA_ACT_NONE && act <= LIA_ACT_GELU_TANH, "lia_gated_act: unknown activation %d", act);
   const unsigned blocks = capped_blocks((size_t)M * F);
-  if (act_f32) gated_act_kernel<float><<<blocks, 256, 0, stream>>>(reinterpret_cast<const float*>(in), ld, up_off, reinterpret_cast<float*>(out), M, F, act);
-  else gated_act_kernel<bf16><<<blocks, 256, 0, stream>>>(reinterpret_cast<const bf16*>(in), ld, up_off, reinterpret_cast<bf16*>(out), M, F, act);
+  if (act_f32) gated_act_kernel<float><<<blocks, 256, 0, stream>>>(reinterpret_cast<const float*>(in), ld, up_off, reinterpret_cast<float*>(out), M, F, act, perm, wt);
+  else gated_act_kernel<bf16><<<blocks, 256, 0, stream>>>(reinterpret_cast<const bf16*>(in), ld, up_off, reinterpret_cast<bf16*>(out), M, F, act, perm, wt);
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }
@@ -472,9 +499,17 @@ extern "C" int lia_router_topk(const float* logits, int* idx, float* wt, int M, 
 
 extern "C" int lia_router_topk_ext(const float* logits, const float* correction, int renorm, int* idx, float* wt, int M, int E, int top,
                                    lia_stream_t stream_) {
+  return lia_router_topk_scored(logits, E, correction, renorm, 0, idx, wt, M, E, top, stream_);
+}
+
+// ldl: row stride of the logits (a row may hold more than the experts' logits); sigmoid != 0: scores are sigmoids, not a softmax
+extern "C" int lia_router_topk_scored(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int* idx, float* wt, int M,
+                                      int E, int top, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
-  LIA_CHECK_ARG(logits && idx && wt && M > 0 && E > 0 && top > 0 && top <= E && E <= 2048, "lia_router_topk: bad arguments (E=%d top=%d)", E, top);
-  router_topk_kernel<<<(M + 3) / 4, 128, (size_t)8 * E * sizeof(float), stream>>>(logits, correction, idx, wt, M, E, top, renorm);
+  LIA_CHECK_ARG(logits && idx && wt && M > 0 && E > 0 && top > 0 && top <= E && E <= 2048 && ldl >= E, "lia_router_topk: bad arguments (E=%d top=%d)", E, top);
+  const size_t smem = (size_t)8 * E * sizeof(float);
+  if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(router_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  router_topk_kernel<<<(M + 3) / 4, 128, smem, stream>>>(logits, ldl, correction, idx, wt, M, E, top, renorm, sigmoid);
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }
@@ -511,6 +546,14 @@ extern "C" int lia_moe_gemm_ext(const void* A, int a_f32, int lda, const void* W
 extern "C" int lia_moe_gemm_act(const void* A, int a_f32, int lda, const void* W, int w_f32, long long w_expert_stride, void* C, int c_f32, int ldc,
                                 const int* perm, const int* tile_expert, int n_tiles, const int* idx, const float* wt, int pairs, int top, int N,
                                 int K, int up, int act, int gated, int n_real, float p0, float p1, lia_stream_t stream_) {
+  return lia_moe_gemm_weighted(A, a_f32, lda, W, w_f32, w_expert_stride, C, c_f32, ldc, perm, tile_expert, n_tiles, idx, wt, pairs, top, N, K, up, act,
+                               gated, n_real, p0, p1, 0, stream_);
+}
+
+// weigh_in != 0: the routing weight multiplies the experts' INPUT (up: act of wt times the sums; down: unweighted)
+extern "C" int lia_moe_gemm_weighted(const void* A, int a_f32, int lda, const void* W, int w_f32, long long w_expert_stride, void* C, int c_f32, int ldc,
+                                     const int* perm, const int* tile_expert, int n_tiles, const int* idx, const float* wt, int pairs, int top, int N,
+                                     int K, int up, int act, int gated, int n_real, float p0, float p1, int weigh_in, lia_stream_t stream_) {
   LIA_CHECK_ARG(act != LIA_ACT_CLAMPED_SWISH || (gated && p0 > 0.f), "lia_moe_gemm: the clamped activation needs the gated form and a positive limit");
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(A && W && C && idx && wt && pairs > 0 && top > 0 && N > 0 && K > 0 && lda >= K && ldc >= N, "lia_moe_gemm: bad arguments");
@@ -521,18 +564,18 @@ extern "C" int lia_moe_gemm_act(const void* A, int a_f32, int lda, const void* W
     LIA_CHECK_ARG(pairs <= 65535, "lia_moe_gemm: too many pairs for the few-rows form");
     dim3 grid((N + 3) / 4, pairs);
     if (a_f32) {
-      if (up) moe_fewrows_kernel<float, float, float, true><<<grid, 128, 0, stream>>>((const float*)A, lda, (const float*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1);
-      else moe_fewrows_kernel<float, float, float, false><<<grid, 128, 0, stream>>>((const float*)A, lda, (const float*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1);
+      if (up) moe_fewrows_kernel<float, float, float, true><<<grid, 128, 0, stream>>>((const float*)A, lda, (const float*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1, weigh_in);
+      else moe_fewrows_kernel<float, float, float, false><<<grid, 128, 0, stream>>>((const float*)A, lda, (const float*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1, weigh_in);
     } else {
-      if (up) moe_fewrows_kernel<bf16, bf16, bf16, true><<<grid, 128, 0, stream>>>((const bf16*)A, lda, (const bf16*)W, w_expert_stride, (bf16*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1);
-      else moe_fewrows_kernel<bf16, bf16, float, false><<<grid, 128, 0, stream>>>((const bf16*)A, lda, (const bf16*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1);
+      if (up) moe_fewrows_kernel<bf16, bf16, bf16, true><<<grid, 128, 0, stream>>>((const bf16*)A, lda, (const bf16*)W, w_expert_stride, (bf16*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1, weigh_in);
+      else moe_fewrows_kernel<bf16, bf16, float, false><<<grid, 128, 0, stream>>>((const bf16*)A, lda, (const bf16*)W, w_expert_stride, (float*)C, ldc, idx, wt, top, N, K, act, gated, n_real, p0, p1, weigh_in);
     }
     LIA_LAUNCH_CHECK();
     return LIA_OK;
   }
   LIA_CHECK_ARG(tile_expert && n_tiles > 0 && n_tiles <= 65535, "lia_moe_gemm: bad tile plan");
   dim3 grid((N + 63) / 64, n_tiles);
-#define LIA_MG(TA, TC, UP_, GATED_) moe_gemm_kernel<TA, TA, TC, UP_, GATED_><<<grid, 256, 0, stream>>>((const TA*)A, lda, (const TA*)W, w_expert_stride, (TC*)C, ldc, perm, tile_expert, wt, top, N, K, act, n_real, p0, p1)
+#define LIA_MG(TA, TC, UP_, GATED_) moe_gemm_kernel<TA, TA, TC, UP_, GATED_><<<grid, 256, 0, stream>>>((const TA*)A, lda, (const TA*)W, w_expert_stride, (TC*)C, ldc, perm, tile_expert, wt, top, N, K, act, n_real, p0, p1, weigh_in)
   if (a_f32) {
     if (up && gated) LIA_MG(float, float, true, true);
     else if (up) LIA_MG(float, float, true, false);
@@ -584,11 +627,20 @@ extern "C" int lia_moe_combine(const void* ypair, int ypair_f32, const int* pos_
 
 extern "C" int lia_moe_combine_ext(const void* ypair, int ypair_f32, const int* pos_of, const float* wt, const void* shared, int act_f32,
                                    const int* idx, int n_real, const void* h, float* y, int M, int W, int top, lia_stream_t stream_) {
+  return lia_moe_combine_gated(ypair, ypair_f32, pos_of, wt, 0, shared, act_f32, nullptr, 0, idx, n_real, h, y, M, W, top, stream_);
+}
+
+// weighted != 0: the experts' outputs carry their routing weights already; shared_gate (fp32, one number per token with row stride
+// ldg, may be null): the shared expert's output is multiplied by its sigmoid
+extern "C" int lia_moe_combine_gated(const void* ypair, int ypair_f32, const int* pos_of, const float* wt, int weighted, const void* shared, int act_f32,
+                                     const float* shared_gate, int ldg, const int* idx, int n_real, const void* h, float* y, int M, int W, int top,
+                                     lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
-  LIA_CHECK_ARG(ypair && y && M > 0 && W > 0 && top > 0 && (!pos_of || wt), "lia_moe_combine: bad arguments");
+  LIA_CHECK_ARG(ypair && y && M > 0 && W > 0 && top > 0 && (!pos_of || wt || weighted), "lia_moe_combine: bad arguments");
+  LIA_CHECK_ARG(!shared_gate || (shared && ldg >= 1), "lia_moe_combine: a gate without a shared expert");
   LIA_CHECK_ARG(!idx || (h && wt && n_real >= 0), "lia_moe_combine: identity experts need the routing weights and the experts' input");
   const unsigned blocks = capped_blocks((size_t)M * W);
-#define LIA_MC(TY, TS) moe_combine_kernel<TY, TS><<<blocks, 256, 0, stream>>>(reinterpret_cast<const TY*>(ypair), pos_of, wt, reinterpret_cast<const TS*>(shared), y, M, W, top, idx, n_real, reinterpret_cast<const TS*>(h))
+#define LIA_MC(TY, TS) moe_combine_kernel<TY, TS><<<blocks, 256, 0, stream>>>(reinterpret_cast<const TY*>(ypair), pos_of, wt, reinterpret_cast<const TS*>(shared), y, M, W, top, idx, n_real, reinterpret_cast<const TS*>(h), weighted, shared_gate, ldg)
   if (ypair_f32 && act_f32) LIA_MC(float, float);
   else if (ypair_f32) LIA_MC(float, bf16);
   else if (act_f32) LIA_MC(bf16, float);

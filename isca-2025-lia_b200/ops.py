@@ -456,19 +456,34 @@ def latent_attn_splits(M, H, max_ctx, sms):
     return max(1, min(want, latent_attn_split_class(max_ctx)))
 
 
-def latent_attn(qa, cache, meta, gate, out, H, kv_rank, rot, scale, max_ctx=0):
-    """Causal softmax attention of every row over its sequence's cached latent rows (csrc/latent_attn.cu).  ``max_ctx``: an
-    upper bound of the rows' history lengths (0: unknown, no split of the keys)."""
+def latent_store(dkv, c_norm_w, meta, cache, kv_rank, eps):
+    """The normalised latent alone into ``cache[slot, pos]`` (designs without a rotated part)."""
+    ldd = _rowmajor(dkv, "dkv")
+    _req(c_norm_w, "c_norm_w", F32); _req(meta, "meta", torch.int32)
+    if cache.dtype != dkv.dtype or not cache.is_contiguous() or cache.shape[2] != kv_rank or dkv.shape[1] != kv_rank or c_norm_w.numel() != kv_rank:
+        raise _lib.LiaError("latent_store: cache must be a contiguous [slots, capacity, kv_rank] tensor of the activations' dtype")
+    check(_lib.load().lia_latent_store(_p(dkv), ldd, _f32(dkv), _p(c_norm_w), _p(meta), _p(cache), cache.stride(0), dkv.shape[0], kv_rank, float(eps),
+                                       _stream()), "lia_latent_store")
+    count_launches()
+
+
+def latent_attn(qa, cache, meta, gate, out, H, kv_rank, rot, scale, max_ctx=0, window=0, sink=None):
+    """Causal softmax attention of every row over its sequence's cached latent rows (csrc/latent_attn.cu), all of them or the last
+    ``window`` (> 0).  ``max_ctx``: an upper bound of the rows' history lengths (0: unknown, no split of the keys).  ``sink`` [H]
+    joins the softmax's denominator."""
     _req(qa, "qa", F32); _req(meta, "meta", torch.int32); _req(out, "out", F32)
-    if gate is not None:
-        _req(gate, "gate", F32)
+    for t, n in ((gate, "gate"), (sink, "sink")):
+        if t is not None:
+            _req(t, n, F32)
     M = qa.shape[0]
-    nsplit = latent_attn_splits(M, H, max_ctx, _sm_count(qa.device))
+    if (sink is not None and sink.numel() != H) or qa.numel() != M * H * (kv_rank + rot) or out.numel() != M * H * kv_rank or cache.shape[2] != kv_rank + rot:
+        raise _lib.LiaError("latent_attn: qa [M, H * (kv_rank + rot)], out [M, H * kv_rank], cache rows of kv_rank + rot, a sink per head")
+    nsplit = latent_attn_splits(M, H, min(max_ctx, window) if window > 0 else max_ctx, _sm_count(qa.device))
     ws = None
     if nsplit > 1:
         ws = torch.empty(_lib.load().lia_latent_attn_workspace_floats(M, H, kv_rank, nsplit), dtype=F32, device=qa.device)
-    check(_lib.load().lia_latent_attn(_p(qa), _p(cache), _f32(cache), cache.stride(0), _p(meta), _p(gate), _p(out), _p(ws), nsplit, M, H,
-                                      kv_rank, rot, float(scale), _stream()), "lia_latent_attn")
+    check(_lib.load().lia_latent_attn_masked(_p(qa), _p(cache), _f32(cache), cache.stride(0), _p(meta), _p(gate), _p(sink), _p(out), _p(ws), nsplit, M, H,
+                                             kv_rank, rot, int(window), float(scale), _stream()), "lia_latent_attn")
     count_launches(2 if nsplit > 1 else 1)
     return out
 
@@ -526,27 +541,38 @@ def ln_gather(x, rows, norm, h, eps):
     return h
 
 
-def gated_act(inp, F, out, act, up_off=-1):
-    """out = act(inp[:, :F]) * inp[:, up_off:up_off + F] (``up_off`` < 0: no second factor)."""
+def gated_act(inp, F, out, act, up_off=-1, perm=None, wt=None):
+    """out = act(inp[:, :F]) * inp[:, up_off:up_off + F] (``up_off`` < 0: no second factor).  ``perm`` and ``wt``: the rows are
+    experts' projections in a plan's order, and both factors are first multiplied by their pair's routing weight."""
     ld = _rowmajor(inp, "inp")
     M = inp.shape[0]
     if tuple(out.shape) != (M, F) or not out.is_contiguous() or out.dtype != inp.dtype:
         raise _lib.LiaError("gated_act: out must be a contiguous [M, F] tensor of the input's dtype")
-    check(_lib.load().lia_gated_act(_p(inp), ld, up_off, _p(out), _f32(out), M, F, act, _stream()), "lia_gated_act")
+    if perm is not None:
+        _req(perm, "perm", I32); _req(wt, "wt", F32)
+        if perm.numel() < M:
+            raise _lib.LiaError("gated_act: the plan's order must cover the rows")
+    check(_lib.load().lia_gated_act_weighted(_p(inp), ld, up_off, _p(out), _f32(out), M, F, act, _p(perm), _p(wt) if perm is not None else None, _stream()),
+          "lia_gated_act")
     count_launches()
     return out
 
 
-def router_topk(logits, top, idx, wt, correction=None, renorm=True):
-    """Softmax over the experts, the ``top`` largest scores and their weights: idx int32 [M, top], wt fp32.  ``correction``
-    [E] is added to the scores for the choice only; ``renorm`` divides the chosen scores by their sum."""
-    _req(logits, "logits", F32); _req(idx, "idx", I32); _req(wt, "wt", F32)
+def router_topk(logits, top, idx, wt, correction=None, renorm=True, sigmoid=False):
+    """Scores of the experts -- a softmax over their logits or (``sigmoid``) the sigmoid of each --, the ``top`` largest and their
+    weights: idx int32 [M, top], wt fp32.  ``correction`` [E] is added to the scores for the choice only; ``renorm`` divides the
+    chosen scores by their sum.  ``logits`` may be the left columns of a wider buffer."""
+    ldl = _rowmajor(logits, "logits")
+    _req(idx, "idx", I32); _req(wt, "wt", F32)
     M, E = logits.shape
+    if logits.dtype != F32:
+        raise _lib.LiaError("router_topk: the logits must be fp32")
     if tuple(idx.shape) != (M, top) or tuple(wt.shape) != (M, top) or (correction is not None and correction.numel() != E):
         raise _lib.LiaError("router_topk: idx and wt must be [M, top], the correction [E]")
     if correction is not None:
         _req(correction, "correction", F32)
-    check(_lib.load().lia_router_topk_ext(_p(logits), _p(correction), int(renorm), _p(idx), _p(wt), M, E, top, _stream()), "lia_router_topk")
+    check(_lib.load().lia_router_topk_scored(_p(logits), ldl, _p(correction), int(renorm), int(sigmoid), _p(idx), _p(wt), M, E, top, _stream()),
+          "lia_router_topk")
     count_launches()
 
 
@@ -562,21 +588,22 @@ def moe_plan(idx, E, perm, tile_expert, pos_of):
     count_launches()
 
 
-def moe_gemm(a, w, out, idx, wt, top, up, act=ACT_NONE, perm=None, tile_expert=None, gated=False, act_params=(0.0, 0.0)):
+def moe_gemm(a, w, out, idx, wt, top, up, act=ACT_NONE, perm=None, tile_expert=None, gated=False, act_params=(0.0, 0.0), weigh_in=False):
     """One projection of every expert over its own rows; ``w`` [E, N, K].  up: out[place] = act(a[token] @ w[e].T);
     down: out[pair] = wt[pair] * a[place] @ w[e].T (fp32).  Without a plan (``perm`` None) a pair's place is the pair.
     ``gated`` (up only): ``w`` is [E, 2N, K], N gate rows then N up rows, and out = act(gate) * up.  Pairs whose expert
     index is E or more (experts without weights) are left out.  ``act_params``: (limit, alpha) of ACT_CLAMPED_SWISH, the gated
-    activation g' sigmoid(alpha g') (u' + 1) on g' = min(g, limit), u' = clamp(u, -limit, limit)."""
+    activation g' sigmoid(alpha g') (u' + 1) on g' = min(g, limit), u' = clamp(u, -limit, limit).  ``weigh_in``: wt multiplies what
+    goes into the expert (the up projection's sums, before the activation) and not what comes out."""
     _dev(a, "a"); _dev(w, "w"); _dev(out, "out")
     E, N, K = w.shape
     if gated:
         N //= 2
     if not (w.is_contiguous() and a.is_contiguous() and out.is_contiguous() and a.shape[1] == K and out.shape[1] == N):
         raise _lib.LiaError(f"moe_gemm: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
-    check(_lib.load().lia_moe_gemm_act(_p(a), _f32(a), K, _p(w), _f32(w), w.stride(0), _p(out), _f32(out), N, _p(perm), _p(tile_expert),
-                                       tile_expert.numel() if tile_expert is not None else 0, _p(idx), _p(wt), idx.numel(), top, N, K, int(up), act,
-                                       int(gated), E, float(act_params[0]), float(act_params[1]), _stream()), "lia_moe_gemm")
+    check(_lib.load().lia_moe_gemm_weighted(_p(a), _f32(a), K, _p(w), _f32(w), w.stride(0), _p(out), _f32(out), N, _p(perm), _p(tile_expert),
+                                            tile_expert.numel() if tile_expert is not None else 0, _p(idx), _p(wt), idx.numel(), top, N, K, int(up), act,
+                                            int(gated), E, float(act_params[0]), float(act_params[1]), int(weigh_in), _stream()), "lia_moe_gemm")
     count_launches()
     return out
 
@@ -606,15 +633,17 @@ def moe_expert_gemms(a, w, out, tiles_per_expert, tile_rows, workspace):
     return out
 
 
-def moe_combine(ypair, shared, y, top, pos_of=None, wt=None, identity=None):
+def moe_combine(ypair, shared, y, top, pos_of=None, wt=None, identity=None, weighted=False, shared_gate=None):
     """y[m] = sum over the token's choices (+ the shared expert's output).  Without a plan ``ypair`` holds the weighted
     outputs pair by pair; with ``pos_of`` and ``wt`` it holds the unweighted outputs in the plan's order.  ``identity`` =
-    (idx, first identity expert, h, wt): a pair routed to an expert from that index on contributes wt * h[m]."""
+    (idx, first identity expert, h, wt): a pair routed to an expert from that index on contributes wt * h[m].  ``weighted``: the
+    outputs in the plan's order carry their weights already (no ``wt``).  ``shared_gate``: an fp32 column [M, 1], the shared expert's output is
+    multiplied by its sigmoid."""
     _dev(ypair, "ypair"); _req(y, "y", F32)
     M, W = y.shape
     if shared is not None and not (shared.is_contiguous() and tuple(shared.shape) == (M, W)):
         raise _lib.LiaError("moe_combine: the shared expert's output must be a contiguous [M, W] tensor")
-    if not ypair.is_contiguous() or ypair.shape[1] != W or (pos_of is None) != (wt is None):
+    if not ypair.is_contiguous() or ypair.shape[1] != W or (pos_of is None or weighted) != (wt is None):
         raise _lib.LiaError("moe_combine: ypair must be a contiguous [.., W] tensor; pos_of and wt go together")
     idx, n_real, h = None, 0, None
     if identity is not None:
@@ -624,8 +653,13 @@ def moe_combine(ypair, shared, y, top, pos_of=None, wt=None, identity=None):
             raise _lib.LiaError("moe_combine: the experts' input must be a contiguous [M, W] tensor of the shared expert's type")
         wt = wt_id
     act = h if h is not None else shared
-    check(_lib.load().lia_moe_combine_ext(_p(ypair), _f32(ypair), _p(pos_of), _p(wt), _p(shared), _f32(act) if act is not None else 1, _p(idx),
-                                          n_real, _p(h), _p(y), M, W, top, _stream()), "lia_moe_combine")
+    ldg = 0
+    if shared_gate is not None:
+        ldg = shared_gate.stride(0)
+        if shared is None or shared_gate.dtype != F32 or tuple(shared_gate.shape) != (M, 1) or not shared_gate.is_cuda:
+            raise _lib.LiaError("moe_combine: the shared expert's gate must be an fp32 [M, 1] column beside a shared expert")
+    check(_lib.load().lia_moe_combine_gated(_p(ypair), _f32(ypair), _p(pos_of), _p(wt), int(weighted), _p(shared), _f32(act) if act is not None else 1,
+                                            _p(shared_gate), ldg, _p(idx), n_real, _p(h), _p(y), M, W, top, _stream()), "lia_moe_combine")
     count_launches()
     return y
 
@@ -955,3 +989,30 @@ def diff_combine(a, out, H, G, vdim, lam, mult, eps):
     check(_lib.load().lia_diff_combine(_p(a), _p(out), _f32(out), M, H, G, vdim, float(lam), float(mult), float(eps), _stream()), "lia_diff_combine")
     count_launches()
     return out
+
+
+# ------------------------------------------------------------------------------------------------------------------
+# Designs whose embedding looks at the token before and whose positions are sine and cosine waves.  (Not in the reference either.)
+# ------------------------------------------------------------------------------------------------------------------
+def embed_bigram_pos(ids, table, meta, x, bigram=None, hashing=None, tokens=None, freq=None, norm_w=None, h=None, eps=0.0):
+    """x[r] = table[id] + bigram[(prev * mul_prev + id * mul_cur) mod buckets] + wave(position) in fp32.  ``hashing`` = (buckets,
+    mul_prev, mul_cur), ``bigram`` [buckets + 1, W] (a sequence's first token takes the last row), ``tokens`` int32 [slots, capacity, 1]
+    the ids of the sequences so far (each row leaves its own there); ``freq`` float64 [(W + 1) // 2]: wave[2i], wave[2i+1] = sin, cos of
+    position * freq[i].  ``h``: the row behind its first norm, norm_w * x / rms(x)."""
+    _req(ids, "ids", torch.int64); _req(x, "x", F32); _req(meta, "meta", I32); _dev(table, "table")
+    rows, W = x.shape
+    buckets, mul_prev, mul_cur = hashing if bigram is not None else (0, 0, 0)
+    if bigram is not None:
+        _req(tokens, "tokens", I32)
+        if bigram.dtype != table.dtype or tuple(bigram.shape) != (buckets + 1, W) or not bigram.is_contiguous() or tokens.dim() != 3 or tokens.shape[2] != 1:
+            raise _lib.LiaError("embed_bigram_pos: bigram must be a contiguous [buckets + 1, W] tensor of the token table's dtype, tokens [slots, capacity, 1]")
+    if freq is not None and (freq.dtype != torch.float64 or not freq.is_cuda or freq.numel() != (W + 1) // 2):
+        raise _lib.LiaError("embed_bigram_pos: freq must be a CUDA float64 tensor of (W + 1) // 2 numbers")
+    if h is not None and (_req(norm_w, "norm_w", F32).numel() != W or not (h.is_cuda and h.is_contiguous() and tuple(h.shape) == (rows, W))):
+        raise _lib.LiaError("embed_bigram_pos: h must be a contiguous [rows, W] tensor, its norm weight fp32 [W]")
+    check(_lib.load().lia_embed_bigram_pos(_p(ids), _p(table), _p(bigram), _f32(table), int(buckets), int(mul_prev), int(mul_cur),
+                                           _p(tokens) if bigram is not None else None, tokens.stride(0) if bigram is not None else 0, _p(freq), _p(meta),
+                                           _p(x), _p(norm_w) if h is not None else None, _p(h), _f32(h) if h is not None else 0, rows, W, table.shape[0],
+                                           float(eps), _stream()), "lia_embed_bigram_pos")
+    count_launches()
+    return x
