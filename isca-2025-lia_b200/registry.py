@@ -37,6 +37,11 @@ def _zatusun():
     return ZatusunForCausalLM
 
 
+def _pazivik():
+    from .modeling_pazivik import PazivikForCausalLM
+    return PazivikForCausalLM
+
+
 register("OPTForCausalLM", _opt)
 register("opt", _opt)
 register("Davasun", _davasun)
@@ -47,6 +52,8 @@ register("Bizetar", _bizetar)
 register("BizetarForCausalLM", _bizetar)
 register("Zatusun", _zatusun)
 register("ZatusunForCausalLM", _zatusun)
+register("Pazivik", _pazivik)
+register("PazivikForCausalLM", _pazivik)
 
 
 def architecture_of(path):

@@ -1,12 +1,13 @@
 """Sequence mixers and feed-forwards that run on a 32-bit residual stream, each with its constants as parameters so that
 any model design can assemble them: a matrix-memory recurrent mixer (mLSTM), attention over a latent key/value cache with
-a partly rotated query/key and an output gate (queries direct or through a latent of their own), linear attention with a fixed
+a partly rotated or unrotated query/key, an output gate, a sliding window and a sink (queries direct or through a latent of their own,
+the cache a layer's own or an earlier layer's), linear attention with a fixed
 decay per head, linear attention with a forget gate per channel, the gated delta rule behind a short convolution, differential
 attention (two softmax maps over shared values, subtracted) under a chunked or sliding mask, sliding-window attention with grouped key/value heads, attention over the whole history with a sink in the
 softmax (behind an optional bias, convolution, norm, temperature and rotation of its inputs, with a distance bias, a blend of
 values across layers and an output gate), and the feed-forwards -- clamped gated, plain gated with any activation, one with a
-polynomial activation between norms, and a routed mixture of experts (plain or gated experts, a shared expert, experts that
-hand the token back).  Each object owns its (fused) weights,
+polynomial activation between norms, and a routed mixture of experts (plain or gated experts weighed on the way out or on the way in, a
+shared expert with or without a gate, experts that hand the token back).  Each object owns its (fused) weights,
 registers its per-sequence state with a ``seq_state.SlotState`` and runs one step over a batch of portions
 (``StepBatch``) through the kernels of ``ops``.
 
@@ -128,12 +129,19 @@ class LatentAttentionMixer:
                       True: channels (2i, 2i+1) turn together, angles from float64 frequencies, ``rot_scaling`` interpolates them
                       (``scaled_rotary_freq``) and sets the amplitude of cos and sin;
       ``gate``        "head": head outputs times sigmoid(Wg h)_h ("g" [H, W]); "channel": the concatenated heads times
-                      sigmoid(Wg h) element by element ("g" [H * vdim, W]); None: no gate."""
+                      sigmoid(Wg h) element by element ("g" [H * vdim, W]); None: no gate;
+      ``rot_dim``     0: queries and keys have no rotated part, the cache row is the latent alone;
+      ``window``      > 0: a position sees only the last ``window`` positions, its own included;
+      ``sink``        True: exp(sink_h) joins the softmax's denominator ("sink" [H]), a term without key or value, not scaled;
+      ``own_latent``  False: the layer makes no latent; its state is an earlier layer's cache, read as it stands (``new_state`` takes
+                      that layer's state), with this layer's own Wq, Wuk, Wuv and window.  Needs ``rot_dim`` = 0."""
 
     def __init__(self, w, heads, dim, rot_dim, vdim, kv_rank, rot_dims, rot_base, scale, norm_eps, dtype, device, q_rank=None, rot_pairs=False,
-                 rot_scaling=None, gate="head"):
+                 rot_scaling=None, gate="head", window=0, sink=False, own_latent=True):
         if gate not in (None, "head", "channel"):
             raise ValueError(f"unknown output gate {gate!r}")
+        if not own_latent and rot_dim:
+            raise ValueError("a layer on another layer's latents has no rotated part")
         if rot_dims % 2 or not 0 <= rot_dims <= rot_dim:
             raise ValueError(f"cannot rotate {rot_dims} of {rot_dim} channels")
         if rot_scaling and not rot_pairs:
@@ -141,32 +149,42 @@ class LatentAttentionMixer:
         self.H, self.dim, self.rot, self.vdim, self.rank = heads, dim, rot_dim, vdim, kv_rank
         self.rot_dims, self.scale, self.eps, self.dtype = rot_dims, float(scale), float(norm_eps), dtype
         self.q_rank, self.gate, self.rot_pairs = q_rank, gate, bool(rot_pairs)
-        stacked = [w["dq"] if q_rank else w["q"], w["dkv"]] + ([w["g"]] if gate == "channel" else [])
+        self.window, self.own_latent = int(window or 0), bool(own_latent)
+        self.sink = w["sink"].to(device=device, dtype=F32).contiguous() if sink else None
+        stacked = [w["dq"] if q_rank else w["q"]] + ([w["dkv"]] if own_latent else []) + ([w["g"]] if gate == "channel" else [])
         self.proj = Linear(stacked, dtype, device)
         if q_rank:
             self.q_norm_w = w["dq.norm"].to(device=device, dtype=F32).contiguous()
             self.up_q = Linear([w["uq"]], dtype, device)
         self.w_gate = w["g"].to(device=device, dtype=dtype).contiguous() if gate == "head" else None
-        self.c_norm_w = w["dkv.norm"].to(device=device, dtype=F32).contiguous()
+        self.c_norm_w = w["dkv.norm"].to(device=device, dtype=F32).contiguous() if own_latent else None
         # Wuk [H*dim, rank] -> per head [rank, dim]: the projection that carries a query into the latent space
         self.w_uk_t = w["uk"].to(device=device, dtype=dtype).view(heads, dim, kv_rank).transpose(1, 2).contiguous()
         self.w_uv = w["uv"].to(device=device, dtype=dtype).contiguous()            # [H*vdim, rank]
         self.out = Linear([w["o"]], dtype, device)
         self.rot_mag = 1.0
-        if self.rot_pairs:
+        if not rot_dim:
+            self.inv_freq = None
+        elif self.rot_pairs:
             f, self.rot_mag = scaled_rotary_freq(rot_dims, rot_base, rot_scaling)
             self.inv_freq = f.to(device).contiguous()                                    # float64
         else:
             self.inv_freq = rotary_inv_freq(rot_dims, rot_base, device)
 
-    def new_state(self, slots):
-        return (slots.add_rows(self.rank + self.rot, self.dtype),)
+    def new_state(self, slots, source=None):
+        """``source``: the state of the layer whose latents this one reads (without a latent of its own)."""
+        if self.own_latent:
+            return (slots.add_rows(self.rank + self.rot, self.dtype),)
+        if source is None or source[0].shape[2] != self.rank:
+            raise ValueError("a layer without a latent of its own needs the state of a layer with latents of the same size")
+        return source
 
     def __call__(self, h, batch, state):
         (cache,) = state
         M, H, D = h.shape[0], self.H, self.rank + self.rot
         y = self.proj(h)
-        q, dkv = self.proj.part(y, 0), self.proj.part(y, 1)
+        q = self.proj.part(y, 0)
+        dkv = self.proj.part(y, 1) if self.own_latent else None
         if self.q_rank:
             cq = torch.empty(M, self.q_rank, dtype=self.dtype, device=h.device)
             ops.rms_norm_rows(q, self.q_norm_w, cq, self.eps)
@@ -176,20 +194,24 @@ class LatentAttentionMixer:
             gate = torch.empty(M, H, dtype=F32, device=h.device)
             ops.linear_small(h, self.w_gate, None, gate, ops.GATE_SIGMOID)
         qa = torch.empty(M, H * D, dtype=F32, device=h.device)
-        ops.latent_prep(q, dkv, self.c_norm_w, self.inv_freq, batch.meta, cache, qa, H, self.dim, self.rot, self.rot_dims, self.rank,
-                        self.eps, pairs=self.rot_pairs, rot_mag=self.rot_mag)
+        if self.rot:
+            ops.latent_prep(q, dkv, self.c_norm_w, self.inv_freq, batch.meta, cache, qa, H, self.dim, self.rot, self.rot_dims, self.rank,
+                            self.eps, pairs=self.rot_pairs, rot_mag=self.rot_mag)
+        elif self.own_latent:
+            ops.latent_store(dkv, self.c_norm_w, batch.meta, cache, self.rank, self.eps)
         # q~[m, h, :rank] = Wuk_h^T q[m, h, :dim]
         ops.linear_plain(q, self.w_uk_t, qa, batch=H, a_batch_stride=self.dim + self.rot, w_batch_stride=self.rank * self.dim,
                          out_batch_stride=D, n=self.rank, k=self.dim)
         lat = torch.empty(M, H * self.rank, dtype=F32, device=h.device)
-        ops.latent_attn(qa, cache, batch.meta, gate, lat, H, self.rank, self.rot, self.scale, batch.max_ctx)
+        ops.latent_attn(qa, cache, batch.meta, gate, lat, H, self.rank, self.rot, self.scale, batch.max_ctx, window=self.window,
+                        sink=self.sink)
         channel = self.gate == "channel"
         o = torch.empty(M, H * self.vdim, dtype=F32 if channel else self.dtype, device=h.device)
         ops.linear_plain(lat, self.w_uv, o, batch=H, a_batch_stride=self.rank, w_batch_stride=self.vdim * self.rank,
                          out_batch_stride=self.vdim, n=self.vdim, k=self.rank)
         if channel:
             og = torch.empty(M, H * self.vdim, dtype=self.dtype, device=h.device)
-            o = ops.sigmoid_mul(o, self.proj.part(y, 2), og)
+            o = ops.sigmoid_mul(o, self.proj.part(y, 2 if self.own_latent else 1), og)
         return self.out(o)
 
 
@@ -587,21 +609,33 @@ class MoEFeedForward:
     ``renorm``; every expert is Wdown act(Wup h), or Wdown (act(Wgate h) * Wup h) when ``experts_w`` carry a "gate"; the last
     ``identity`` router outputs are experts without weights that hand the token back; ``act`` = ops.ACT_CLAMPED_SWISH with
     ``act_params`` = (limit, alpha) makes a gated expert Wdown (g' sigmoid(alpha g') (u' + 1)), g' = min(Wgate h, limit), u' = clamp(Wup h, +-limit);
-    with ``renorm`` the weights equal a softmax restricted to the selected experts' logits; a shared expert (optional) runs for
-    every token and is added.  ``experts_w``: list of {"up", "down"[, "gate"]} per expert.  The (token, choice) pairs are
+    with ``renorm`` the weights equal a softmax restricted to the selected experts' logits; ``score`` = "sigmoid": an expert's score is
+    the sigmoid of its logit; ``weigh`` = "input": the weight multiplies what goes into the expert (expert(w * h)) instead of what
+    comes out; a shared expert (optional) runs for every token and is added, times sigmoid(``shared_gate`` h) if that weight [1, W] is
+    given (its logit rides on the router's projection).  ``experts_w``: list of {"up", "down"[, "gate"]} per expert.  The (token, choice) pairs are
     grouped by expert on the device (no host round trip) and each projection runs as one grouped launch; a handful of pairs
     (decoding) take the form with one warp per output instead.  The result is fp32."""
 
     FEW_PAIRS = 48            # up to here: one warp per output, no plan
     TENSOR_CORE_PAIRS = 512   # from here (bf16, sizes that are multiples of 8): every expert's rows through the tensor-core GEMM
 
-    def __init__(self, router_w, experts_w, top, ff, act, shared, dtype, device, correction=None, renorm=True, identity=0, act_params=(0.0, 0.0)):
+    def __init__(self, router_w, experts_w, top, ff, act, shared, dtype, device, correction=None, renorm=True, identity=0, act_params=(0.0, 0.0),
+                 score="softmax", weigh="output", shared_gate=None):
+        if score not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
+            raise ValueError(f"unknown option: score={score!r} weigh={weigh!r}")
+        if shared_gate is not None and shared is None:
+            raise ValueError("a gate without a shared expert")
+        if weigh == "input" and act == ops.ACT_CLAMPED_SWISH:
+            raise ValueError("the clamped activation weighs an expert's output")
+        self.sigmoid, self.weigh_in, self.shared_gated = score == "sigmoid", weigh == "input", shared_gate is not None
         self.E, self.top, self.ff, self.act, self.dtype = len(experts_w), int(top), ff, act, dtype
         self.act_params = (float(act_params[0]), float(act_params[1]))      # ACT_CLAMPED_SWISH (gated experts): (limit, alpha)
         self.identity, self.renorm = int(identity), bool(renorm)
         self.R = self.E + self.identity                          # router outputs
         if not 1 <= self.top <= self.R or self.E < 1 or router_w.shape[0] != self.R:
             raise ValueError(f"top = {top} of {self.E} experts + {self.identity} identity experts, router of {router_w.shape[0]} outputs")
+        if shared_gate is not None:
+            router_w = torch.cat([router_w, shared_gate], 0)     # one launch: the experts' logits, then the shared expert's
         self.router = router_w.to(device=device, dtype=dtype).contiguous()
         self.correction = correction.to(device=device, dtype=F32).contiguous() if correction is not None else None
         self.gated = "gate" in experts_w[0]
@@ -621,7 +655,7 @@ class MoEFeedForward:
             ws = Linear._gemm_ws[key] = ops.GemmWorkspace(need, device)
         return ws
 
-    def _experts_tensor_core(self, h, idx, wt, y):
+    def _experts_tensor_core(self, h, idx, wt, y, shared_gate):
         """Prompts: the pairs grouped by expert (tiles of 64 rows), the rows gathered into that order, then one tensor-core
         GEMM per expert and projection on its contiguous rows (launched back to back from the library).  The tile table comes to the host once per call (the only
         round trip; decode steps never take this path, so they stay capturable)."""
@@ -646,10 +680,10 @@ class MoEFeedForward:
             if self.act == ops.ACT_CLAMPED_SWISH:
                 ops.clamped_glu(up, ff, ff, mid, *self.act_params)
             else:
-                ops.gated_act(up, ff, mid, self.act, up_off=ff if self.gated else -1)
+                ops.gated_act(up, ff, mid, self.act, up_off=ff if self.gated else -1, perm=perm if self.weigh_in else None, wt=wt)
             ops.moe_expert_gemms(mid, self.w_down, ys, counts, tm, self._workspace(rows, W, ff, dev))
-        ops.moe_combine(ys, self.shared(h) if self.shared is not None else None, y, top, pos_of=pos_of, wt=wt,
-                        identity=(idx, E, h, wt) if self.identity else None)
+        ops.moe_combine(ys, self.shared(h) if self.shared is not None else None, y, top, pos_of=pos_of, wt=None if self.weigh_in else wt,
+                        identity=(idx, E, h, wt) if self.identity else None, weighted=self.weigh_in, shared_gate=shared_gate)
         return y
 
     def __call__(self, h, router_input=None):
@@ -657,21 +691,22 @@ class MoEFeedForward:
         router logits that do not see that rounding; None: the router reads ``h``."""
         M, W, dev = h.shape[0], h.shape[1], h.device
         R, top = self.R, self.top
-        logits = torch.empty(M, R, dtype=F32, device=dev)
+        logits = torch.empty(M, R + self.shared_gated, dtype=F32, device=dev)
         ops.linear_small(h if router_input is None else router_input, self.router, None, logits, ops.GATE_NONE)
         idx = torch.empty(M, top, dtype=torch.int32, device=dev)
         wt = torch.empty(M, top, dtype=F32, device=dev)
-        ops.router_topk(logits, top, idx, wt, correction=self.correction, renorm=self.renorm)
+        ops.router_topk(logits[:, :R], top, idx, wt, correction=self.correction, renorm=self.renorm, sigmoid=self.sigmoid)
+        shared_gate = logits[:, R:] if self.shared_gated else None
         identity = (idx, self.E, h, wt) if self.identity else None
         pairs = M * top
         y = torch.empty(M, W, dtype=F32, device=dev)
         if self.tensor_core and pairs >= self.TENSOR_CORE_PAIRS and h.is_contiguous() and not torch.cuda.is_current_stream_capturing():
-            return self._experts_tensor_core(h, idx, wt, y)
+            return self._experts_tensor_core(h, idx, wt, y, shared_gate)
         ypair = torch.empty(pairs, W, dtype=F32, device=dev)
         if pairs <= self.FEW_PAIRS:
             mid = torch.empty(pairs, self.ff, dtype=self.dtype, device=dev)
-            ops.moe_gemm(h, self.w_up, mid, idx, wt, top, True, self.act, gated=self.gated, act_params=self.act_params)
-            ops.moe_gemm(mid, self.w_down, ypair, idx, wt, top, False)
+            ops.moe_gemm(h, self.w_up, mid, idx, wt, top, True, self.act, gated=self.gated, act_params=self.act_params, weigh_in=self.weigh_in)
+            ops.moe_gemm(mid, self.w_down, ypair, idx, wt, top, False, weigh_in=self.weigh_in)
         else:
             n_tiles, tm = ops.moe_tiles(pairs, R)
             perm = torch.empty(n_tiles * tm, dtype=torch.int32, device=dev)
@@ -679,7 +714,8 @@ class MoEFeedForward:
             pos_of = torch.empty(pairs, dtype=torch.int32, device=dev)
             ops.moe_plan(idx, R, perm, tile_expert, pos_of)
             mid = torch.empty(n_tiles * tm, self.ff, dtype=self.dtype, device=dev)
-            ops.moe_gemm(h, self.w_up, mid, idx, wt, top, True, self.act, perm, tile_expert, gated=self.gated, act_params=self.act_params)
-            ops.moe_gemm(mid, self.w_down, ypair, idx, wt, top, False, ops.ACT_NONE, perm, tile_expert)
-        ops.moe_combine(ypair, self.shared(h) if self.shared is not None else None, y, top, identity=identity)
+            ops.moe_gemm(h, self.w_up, mid, idx, wt, top, True, self.act, perm, tile_expert, gated=self.gated, act_params=self.act_params,
+                         weigh_in=self.weigh_in)
+            ops.moe_gemm(mid, self.w_down, ypair, idx, wt, top, False, ops.ACT_NONE, perm, tile_expert, weigh_in=self.weigh_in)
+        ops.moe_combine(ypair, self.shared(h) if self.shared is not None else None, y, top, identity=identity, shared_gate=shared_gate)
         return y
