@@ -6,6 +6,8 @@ attention mixers on a 32-bit residual stream).
 key/value heads on the same attention kernel, dense and mixture-of-experts feed-forwards, step-served).
 `bench.py --compare-zatusun`: the same for Zatusun beside Bebulorn, the closest existing model (a matrix-state recurrence, masked
 softmax attention and routed experts on the same kernels, a looped block, step-served).
+`bench.py --compare-pazivik`: the same for Pazivik beside Zatusun, the closest existing model (latent attention on the same kernel,
+gated routed experts, pre-norm fp32 stream, step-served).
 
 Each operation of ``ops`` is wrapped for the duration of an instrumented pass: CUDA events around the call, and the
 operation's algorithmic FLOPs and bytes from its arguments.  roofline time = max(FLOPs / peak, bytes / HBM bandwidth)
@@ -49,8 +51,15 @@ def _cost(name, a, kw):
         return 4.0 * M * H * dim * vdim, state + M * H * (2 * dim + vdim) * q.element_size() + _nbytes(o), "f32"
     if name == "latent_attn":
         qa, cache, meta, out, H, rank, rot = a[0], a[1], a[2], a[4], a[5], a[6], a[7]
-        keys = float(kw.get("_keys", 0))                                           # sum over rows of visible keys
-        return 2.0 * keys * H * (2 * rank + rot), _nbytes(qa, out) + kw.get("_ctx", 0) * (rank + rot) * cache.element_size(), "f32"
+        win = kw.get("window", 0) > 0
+        keys = float(kw.get("_wkeys" if win else "_keys", 0))                      # sum over rows of visible keys
+        return 2.0 * keys * H * (2 * rank + rot), _nbytes(qa, out) + kw.get("_wctx" if win else "_ctx", 0) * (rank + rot) * cache.element_size(), "f32"
+    if name == "latent_store":
+        dkv, cache = a[0], a[3]
+        return 0.0, _nbytes(dkv) + dkv.numel() * cache.element_size(), "mem"
+    if name == "embed_bigram_pos":
+        table, x, h = a[1], a[3], kw.get("h")
+        return 0.0, 2.0 * x.numel() * table.element_size() + _nbytes(x, h), "mem"
     if name == "linear_scan":
         q, S, segs, H, G, dim, vdim, o = a[0], a[3], a[4], a[5], a[6], a[7], a[8], a[9]
         M = q.shape[0]
@@ -105,7 +114,8 @@ class Instrument:
              "rms_add_norm", "embed_rmsnorm", "rms_gather", "layernorm", "attn_prefill", "attn_decode", "embed", "argmax", "argmax_f32",
              "linear_scan", "conv_prep", "conv_state_update", "kv_store", "window_attn", "ln_add_norm", "embed_rows", "ln_gather", "gated_act",
              "router_topk", "moe_plan", "moe_gemm", "moe_gather", "moe_expert_gemms", "moe_combine", "qkv_prep", "gated_rms_add", "poly_norm",
-             "embed_scale_pos", "residual_norm", "rms_norm_rows", "sigmoid_mul", "softcap", "forget_gate_prep", "forget_scan", "diff_combine")
+             "embed_scale_pos", "residual_norm", "rms_norm_rows", "sigmoid_mul", "softcap", "forget_gate_prep", "forget_scan", "diff_combine",
+             "latent_store", "embed_bigram_pos")
 
     def __init__(self):
         self.records, self.saved, self.extra = [], {}, {}
@@ -218,10 +228,24 @@ def zatusun_config(width, n_runs):
             "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5}, "logit_softcap": 30.0}
 
 
+def pazivik_config(width, n_layers):
+    """Layer sizes of a ~1-3 B model: latent attention with heads of 128 query/key and 128 value channels, a 512-wide latent and a
+    window of 1024; every second layer reads the latents of the one before it; feed-forwards alternate between a dense 2.75 x one
+    and 16 gated experts of 0.6875 x (2 chosen) with a shared expert of the same size."""
+    H = width // 128
+    ff = width * 11 // 16
+    dense = {"kind": "dense", "ff": width * 11 // 4}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": ff}, "shared": {"ff": ff}}
+    base = {"heads": H, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5, "mask": {"size": 1024}}
+    layers = [{"type": "latent_attention", "mixer": dict(base, kv_from=i - 1) if i % 2 else dict(base), "mlp": moe if i % 2 else dense} for i in range(n_layers)]
+    return {"architecture": "Pazivik", "vocab": 32000, "width": width, "layers": layers, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}}
+
+
 def _window_keys(layers, n_new, ctx_before):
     """Sum over the new rows of the keys inside the first attention layer's window (the whole history where a layer names
     none), and the cached rows those windows span."""
-    first = next((l for l in layers if l["type"].startswith("attention")), None)
+    first = next((l for l in layers if l["type"].startswith("attention") or (l["type"] == "latent_attention" and "mask" in l["mixer"])), None)
     win = first["mixer"].get("mask", {}).get("size", 1 << 30) if first else 0
     if not win:
         return 0, 0
@@ -302,6 +326,27 @@ def run_zatusun(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=204
         rec = {"width": width, "layers": n_layers, "prompt": prompt, "decode_context": decode_ctx}
         for name, make in (("zatusun", lambda: ZatusunForCausalLM(ZatusunConfig.from_dict(zatusun_config(width, n_layers)), dev, BF16)),
                            ("bebulorn", lambda: BebulornForCausalLM(BebulornConfig.from_dict(bebulorn_config(width, n_layers)), dev, BF16))):
+            m = make().init_weights(seed=1)
+            rec[name] = step_model(m, m.config, pk, g, prompt, decode_ctx, decode_batches, new)
+            del m
+            torch.cuda.empty_cache()
+        out["sizes"].append(rec)
+    return out
+
+
+def run_pazivik(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=2048, decode_batches=(1, 16), new=16):
+    """Pazivik beside Zatusun at equal width and number of layer runs."""
+    from .modeling_pazivik import PazivikConfig, PazivikForCausalLM
+    from .modeling_zatusun import ZatusunConfig, ZatusunForCausalLM
+    dev = torch.device("cuda", 0)
+    props = torch.cuda.get_device_properties(dev)
+    pk = dict(pk, fp32_nominal_tflops=props.multi_processor_count * 128 * 2 * 1.965e9 / 1e12)
+    out = {"peaks": pk, "sizes": []}
+    g = torch.Generator().manual_seed(0)
+    for width in widths:
+        rec = {"width": width, "layers": n_layers, "prompt": prompt, "decode_context": decode_ctx}
+        for name, make in (("pazivik", lambda: PazivikForCausalLM(PazivikConfig.from_dict(pazivik_config(width, n_layers)), dev, BF16)),
+                           ("zatusun", lambda: ZatusunForCausalLM(ZatusunConfig.from_dict(zatusun_config(width, n_layers)), dev, BF16))):
             m = make().init_weights(seed=1)
             rec[name] = step_model(m, m.config, pk, g, prompt, decode_ctx, decode_batches, new)
             del m

@@ -372,7 +372,7 @@ def linear_plain(a, w, out, scale=1.0, batch=1, a_batch_stride=0, w_batch_stride
     M = a.shape[0]
     K = k if k is not None else a.shape[1]
     N = n if n is not None else out.shape[1]
-    ldw = w.stride(-2) if w.dim() >= 2 else K
+    ldw = w.stride(-2) if w.dim() >= 2 and w.shape[-2] > 1 else max(K, w.shape[-1])     # (a single row's stride may be anything)
     if out.shape[0] != M:
         raise _lib.LiaError("linear_plain: a and out differ in rows")
     check(_lib.load().lia_linear_plain(_p(a), _f32(a), lda, a_batch_stride, _p(w), _f32(w), ldw, w_batch_stride, _p(out), _f32(out), ldc,

@@ -29,10 +29,11 @@ def _pad8(n):
 
 class StepBatch:
     """The token rows of one step: ``segs`` int32 [n, 4] = (slot, first position, first row, rows) per portion and
-    ``meta`` int32 [rows, 2] = (slot, position) per row, both on the device."""
+    ``meta`` int32 [rows, 2] = (slot, position) per row, both on the device; ``portions``: the numbers of ``segs`` on the host
+    (None: not known there)."""
 
-    def __init__(self, rows, segs, meta, max_ctx=0):
-        self.rows, self.segs, self.meta = rows, segs, meta
+    def __init__(self, rows, segs, meta, max_ctx=0, portions=None):
+        self.rows, self.segs, self.meta, self.portions = rows, segs, meta, portions
         self.max_ctx = max_ctx              # longest history (tokens cached after this step) among the step's sequences
         self.scratch = {}                   # what one layer of this step leaves for later layers (per-token tensors)
 
@@ -123,7 +124,9 @@ class LatentAttentionMixer:
     """Attention over a latent cache: per token one normalised latent (kv_rank) and one rotated key part (rot_dim) shared by
     the heads are cached; head h's unrotated key and value are Wuk_h c and Wuv_h c.  Queries are laid out per head as
     [dim unrotated | rot_dim rotated]; causal softmax with ``scale``; then Wo.  The kernels work in the latent space
-    (csrc/latent_attn.cu), so Wuk is applied to the query and Wuv to the attention's output.  Options:
+    (csrc/latent_attn.cu), so Wuk is applied to the query and Wuv to the attention's output.  A long portion of a sequence, whose rows
+    share their keys, takes the other order where that is less work (``_expand``): Wuk and Wuv are applied once to the latents
+    it sees, and the rows attend to plain per-head keys and values (csrc/window_attn.cu).  Options:
       ``q_rank``      None: q = Wq h ("q"); a number: q = Wuq RMSnorm(Wdq h) with the plain weight "dq.norm" ("dq", "uq");
       ``rot_pairs``   False: rotary "rotate half" over the first ``rot_dims`` channels of the rotated part (fp32 angles);
                       True: channels (2i, 2i+1) turn together, angles from float64 frequencies, ``rot_scaling`` interpolates them
@@ -135,6 +138,9 @@ class LatentAttentionMixer:
       ``sink``        True: exp(sink_h) joins the softmax's denominator ("sink" [H]), a term without key or value, not scaled;
       ``own_latent``  False: the layer makes no latent; its state is an earlier layer's cache, read as it stands (``new_state`` takes
                       that layer's state), with this layer's own Wq, Wuk, Wuv and window.  Needs ``rot_dim`` = 0."""
+
+    EXPAND_ROWS = 64          # portions of at least this many rows may expand the latents they see ...
+    EXPAND_RATIO = 4          # ... if these are at most this many times the rows
 
     def __init__(self, w, heads, dim, rot_dim, vdim, kv_rank, rot_dims, rot_base, scale, norm_eps, dtype, device, q_rank=None, rot_pairs=False,
                  rot_scaling=None, gate="head", window=0, sink=False, own_latent=True):
@@ -161,6 +167,10 @@ class LatentAttentionMixer:
         # Wuk [H*dim, rank] -> per head [rank, dim]: the projection that carries a query into the latent space
         self.w_uk_t = w["uk"].to(device=device, dtype=dtype).view(heads, dim, kv_rank).transpose(1, 2).contiguous()
         self.w_uv = w["uv"].to(device=device, dtype=dtype).contiguous()            # [H*vdim, rank]
+        self.up_k = self.up_v = None
+        if not rot_dim and gate is None and dim + vdim < 2 * kv_rank and max(dim, vdim) <= 512:
+            self.up_k, self.up_v = Linear([w["uk"]], dtype, device), Linear([w["uv"]], dtype, device)
+            self.w_uv = self.up_v.weight
         self.out = Linear([w["o"]], dtype, device)
         self.rot_mag = 1.0
         if not rot_dim:
@@ -193,26 +203,62 @@ class LatentAttentionMixer:
         if self.gate == "head":
             gate = torch.empty(M, H, dtype=F32, device=h.device)
             ops.linear_small(h, self.w_gate, None, gate, ops.GATE_SIGMOID)
-        qa = torch.empty(M, H * D, dtype=F32, device=h.device)
+        channel = self.gate == "channel"
+        o = torch.empty(M, H * self.vdim, dtype=F32 if channel else self.dtype, device=h.device)
+        qa = None
         if self.rot:
+            qa = torch.empty(M, H * D, dtype=F32, device=h.device)
             ops.latent_prep(q, dkv, self.c_norm_w, self.inv_freq, batch.meta, cache, qa, H, self.dim, self.rot, self.rot_dims, self.rank,
                             self.eps, pairs=self.rot_pairs, rot_mag=self.rot_mag)
         elif self.own_latent:
             ops.latent_store(dkv, self.c_norm_w, batch.meta, cache, self.rank, self.eps)
-        # q~[m, h, :rank] = Wuk_h^T q[m, h, :dim]
-        ops.linear_plain(q, self.w_uk_t, qa, batch=H, a_batch_stride=self.dim + self.rot, w_batch_stride=self.rank * self.dim,
-                         out_batch_stride=D, n=self.rank, k=self.dim)
-        lat = torch.empty(M, H * self.rank, dtype=F32, device=h.device)
-        ops.latent_attn(qa, cache, batch.meta, gate, lat, H, self.rank, self.rot, self.scale, batch.max_ctx, window=self.window,
-                        sink=self.sink)
-        channel = self.gate == "channel"
-        o = torch.empty(M, H * self.vdim, dtype=F32 if channel else self.dtype, device=h.device)
-        ops.linear_plain(lat, self.w_uv, o, batch=H, a_batch_stride=self.rank, w_batch_stride=self.vdim * self.rank,
-                         out_batch_stride=self.vdim, n=self.vdim, k=self.rank)
+        done = 0                                          # rows before this one have their output
+        for i, (slot, p0, row, n) in enumerate(batch.portions if self.up_k is not None and batch.portions is not None else ()):
+            base = max(0, p0 - self.window + 1) if self.window else 0
+            if n >= self.EXPAND_ROWS and p0 + n - base <= self.EXPAND_RATIO * n:
+                self._in_latent_space(q, qa, cache, gate, batch, o, done, row)
+                self._expand(q[row:row + n], cache[slot, base:p0 + n], self._positions_from(batch, i, base), p0 + n - base, o[row:row + n])
+                done = row + n
+        self._in_latent_space(q, qa, cache, gate, batch, o, done, M)
         if channel:
             og = torch.empty(M, H * self.vdim, dtype=self.dtype, device=h.device)
             o = ops.sigmoid_mul(o, self.proj.part(y, 2 if self.own_latent else 1), og)
         return self.out(o)
+
+    def _in_latent_space(self, q, qa, cache, gate, batch, o, r0, r1):
+        """Rows [r0, r1) of ``o``: the query carried into the latent space, attention there, Wuv on what comes out."""
+        n, H, D = r1 - r0, self.H, self.rank + self.rot
+        if n <= 0:
+            return
+        q, o, meta = q[r0:r1], o[r0:r1], batch.meta[r0:r1]
+        gate = gate[r0:r1] if gate is not None else None
+        qa = torch.empty(n, H * D, dtype=F32, device=o.device) if qa is None else qa[r0:r1]
+        # q~[m, h, :rank] = Wuk_h^T q[m, h, :dim]
+        ops.linear_plain(q, self.w_uk_t, qa, batch=H, a_batch_stride=self.dim + self.rot, w_batch_stride=self.rank * self.dim,
+                         out_batch_stride=D, n=self.rank, k=self.dim)
+        lat = torch.empty(n, H * self.rank, dtype=F32, device=o.device)
+        ops.latent_attn(qa, cache, meta, gate, lat, H, self.rank, self.rot, self.scale, batch.max_ctx, window=self.window, sink=self.sink)
+        ops.linear_plain(lat, self.w_uv, o, batch=H, a_batch_stride=self.rank, w_batch_stride=self.vdim * self.rank,
+                         out_batch_stride=self.vdim, n=self.vdim, k=self.rank)
+
+    def _expand(self, q, latents, meta, ctx, o):
+        """One portion's output rows ``o``: per-head keys and values of the ``latents`` [ctx, rank] it sees (as they are cached), then
+        attention over those; ``meta``: the rows as (0, position among the latents)."""
+        H = self.H
+        k, v = self.up_k(latents), self.up_v(latents)
+        ops.window_attn(q, k.unsqueeze(0), v.unsqueeze(0), meta, None, o, H, H, self.dim, self.vdim, self.window, self.scale, 0.0, nseg=1, max_ctx=ctx,
+                        sink=self.sink)
+
+    @staticmethod
+    def _positions_from(batch, i, base):
+        """(0, position - base) of the rows of portion ``i``, shared by the step's layers."""
+        key = ("positions from", i, base)
+        if key not in batch.scratch:
+            _, _, row, n = batch.portions[i]
+            rel = torch.zeros(n, 2, dtype=torch.int32, device=batch.meta.device)
+            torch.sub(batch.meta[row:row + n, 1], base, out=rel[:, 1])
+            batch.scratch[key] = rel
+        return batch.scratch[key]
 
 
 class ClampedGLU:
