@@ -122,23 +122,6 @@ __global__ void __launch_bounds__(128) latent_prep_pairs_kernel(const T* __restr
   }
 }
 
-// cache[slot][pos] = cw * d / sqrt(mean(d^2) + eps) over the row's kv_rank numbers; one warp per token row
-template <typename T>
-__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ dkv, int ldd, const float* __restrict__ cw, const int* __restrict__ meta,
-                                                           T* __restrict__ cache, long long slot_stride, int M, int kv_rank, float eps) {
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= M) return;
-  const T* d = dkv + (size_t)row * ldd;
-  T* crow = cache + (size_t)meta[2 * row] * slot_stride + (size_t)meta[2 * row + 1] * kv_rank;
-  float ss = 0.f;
-  for (int i = lane; i < kv_rank; i += 32) {
-    const float v = ldf(d + i);
-    ss += v * v;
-  }
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)kv_rank + eps);
-  for (int i = lane; i < kv_rank; i += 32) stf(crow + i, ldf(d + i) * inv * cw[i]);
-}
-
 constexpr int TK = 32;     // cached rows per stage (= one warp's lanes: lane j scores key j)
 constexpr int HG = 8;      // heads per block (= warps per block: warp w scores head w)
 
@@ -152,6 +135,52 @@ __device__ __forceinline__ void load_vec(const float* p, float* f) {
 }
 template <typename T> struct Vec { static constexpr int N = 8; };
 template <> struct Vec<float> { static constexpr int N = 4; };
+__device__ __forceinline__ void store_vec(bf16* p, const float* f) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+}
+__device__ __forceinline__ void store_vec(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+
+// cache[slot][pos] = cw * d / sqrt(mean(d^2) + eps) over the row's kv_rank numbers; one warp per token row.  `vec`: rows and
+// cache rows allow 128-bit accesses, and a row of at most 4 vectors per lane stays in registers between the sum and the store.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ dkv, int ldd, const float* __restrict__ cw, const int* __restrict__ meta,
+                                                           T* __restrict__ cache, long long slot_stride, int M, int kv_rank, float eps, int vec) {
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= M) return;
+  const T* d = dkv + (size_t)row * ldd;
+  T* crow = cache + (size_t)meta[2 * row] * slot_stride + (size_t)meta[2 * row + 1] * kv_rank;
+  float ss = 0.f;
+  if (vec) {
+    constexpr int N = Vec<T>::N;
+    float v[4][N];
+#pragma unroll
+    for (int s = 0; s < 4; ++s) {
+      const int i = (s * 32 + lane) * N;
+      if (i < kv_rank) {
+        load_vec(d + i, v[s]);
+#pragma unroll
+        for (int j = 0; j < N; ++j) ss += v[s][j] * v[s][j];
+      }
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)kv_rank + eps);
+#pragma unroll
+    for (int s = 0; s < 4; ++s) {
+      const int i = (s * 32 + lane) * N;
+      if (i < kv_rank) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[s][j] *= inv * cw[i + j];
+        store_vec(crow + i, v[s]);
+      }
+    }
+    return;
+  }
+  for (int i = lane; i < kv_rank; i += 32) {
+    const float v = ldf(d + i);
+    ss += v * v;
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)kv_rank + eps);
+  for (int i = lane; i < kv_rank; i += 32) stf(crow + i, ldf(d + i) * inv * cw[i]);
+}
 
 // 1 / the softmax's denominator for sums taken relative to the maximum m; a sink joins with exp(sink - m), and where it is the
 // larger one everything is taken relative to the sink instead (exp(sink - m) may overflow)
@@ -434,12 +463,15 @@ extern "C" int lia_latent_store(const void* dkv, int ldd, int act_f32, const flo
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(dkv && c_norm_w && meta && cache && M > 0 && kv_rank > 0 && ldd >= kv_rank, "lia_latent_store: bad arguments");
   const unsigned grid = (unsigned)((M + 3) / 4);
+  const int n = act_f32 ? Vec<float>::N : Vec<bf16>::N;
+  const int vec = kv_rank % n == 0 && kv_rank <= 4 * 32 * n && ldd % n == 0 && slot_stride % n == 0 && reinterpret_cast<uintptr_t>(dkv) % 16 == 0 &&
+                  reinterpret_cast<uintptr_t>(cache) % 16 == 0;
   if (act_f32)
     latent_store_kernel<float><<<grid, 128, 0, stream>>>(reinterpret_cast<const float*>(dkv), ldd, c_norm_w, meta, reinterpret_cast<float*>(cache),
-                                                         slot_stride, M, kv_rank, eps);
+                                                         slot_stride, M, kv_rank, eps, vec);
   else
     latent_store_kernel<bf16><<<grid, 128, 0, stream>>>(reinterpret_cast<const bf16*>(dkv), ldd, c_norm_w, meta, reinterpret_cast<bf16*>(cache),
-                                                        slot_stride, M, kv_rank, eps);
+                                                        slot_stride, M, kv_rank, eps, vec);
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }

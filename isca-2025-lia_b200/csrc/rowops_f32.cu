@@ -143,17 +143,22 @@ __global__ void __launch_bounds__(256) embed_bigram_pos_kernel(const int64_t* __
     if (threadIdx.x == 0) tokens[(size_t)slot * token_stride + p] = (int)id;
   }
   float ss = 0.f;
-  for (int i = threadIdx.x; i < W; i += 256) {
-    float v = ldf(e + i);
-    if (b != nullptr) v += ldf(b + i);
+  for (int k = threadIdx.x; 2 * k < W; k += 256) {          // a thread takes both channels of one wave
+    float wave[2] = {0.f, 0.f};
     if (freq != nullptr) {
-      const double a = (double)p * freq[i >> 1];
-      const float r = (float)(a - rint(a * 0.15915494309189533577) * 6.28318530717958647693);
-      v += (i & 1) ? cosf(r) : sinf(r);
+      const double a = (double)p * freq[k];
+      sincosf((float)(a - rint(a * 0.15915494309189533577) * 6.28318530717958647693), &wave[0], &wave[1]);
     }
-    x[(size_t)row * W + i] = v;
-    xs[i] = v;
-    ss += v * v;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = 2 * k + j;
+      if (i < W) {
+        const float v = ldf(e + i) + (b != nullptr ? ldf(b + i) : 0.f) + wave[j];
+        x[(size_t)row * W + i] = v;
+        xs[i] = v;
+        ss += v * v;
+      }
+    }
   }
   if (h == nullptr) return;
   ss = block_sum<256>(ss, red);

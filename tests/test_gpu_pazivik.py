@@ -93,15 +93,16 @@ def test_embedding_with_bigram_and_waves(W):
     assert torch.equal(x2.cpu(), table[first[:3]])
 
 
-@pytest.mark.parametrize("rank", [17, 40, 264])
-def test_latent_store(rank):
+@pytest.mark.parametrize("rank,at", [(17, 5), (40, 5), (40, 8), (264, 8), (512, 16), (1024, 0), (1032, 8)])
+def test_latent_store(rank, at):
+    """Column slices that allow 128-bit accesses and slices that do not, rows that fit a warp's registers and longer ones."""
     g = gen(1)
-    y, w = torch.randn(70, rank + 13, generator=g) * 3.0, 1.0 + 0.3 * torch.randn(rank, generator=g)
+    y, w = torch.randn(70, rank + 24, generator=g) * 3.0, 1.0 + 0.3 * torch.randn(rank, generator=g)
     for dt, tol in ((F32, 2e-6), (BF16, 5e-3)):
         yy = y.to(dt)
         cache = torch.zeros(3, 80, rank, dtype=dt, device=DEV)
-        ops.latent_store(yy.to(DEV)[:, 5:5 + rank], w.to(DEV), make_batch([(2, 10, 69), (0, 79, 1)]).meta, cache, rank, 1e-6)
-        want = O.rms_norm(yy.double()[:, 5:5 + rank], w.double(), 1e-6)
+        ops.latent_store(yy.to(DEV)[:, at:at + rank], w.to(DEV), make_batch([(2, 10, 69), (0, 79, 1)]).meta, cache, rank, 1e-6)
+        want = O.rms_norm(yy.double()[:, at:at + rank], w.double(), 1e-6)
         assert rel(cache[2, 10:79], want[:69]) < tol and rel(cache[0, 79], want[69]) < tol
         assert not cache[1].any() and not cache[2, :10].any() and not cache[2, 79].any() and not cache[0, :79].any()
 
