@@ -32,7 +32,7 @@
 extern "C" {
 #endif
 
-#define LIA_ABI_VERSION 10
+#define LIA_ABI_VERSION 11
 
 typedef void* lia_stream_t; /* cudaStream_t */
 
@@ -307,7 +307,8 @@ int lia_latent_attn(const float* qa, const void* cache, int cache_f32, long long
  * with grouped key/value heads, and dense or mixture-of-experts feed-forwards.  Same conventions as the section above.
  * The reference has none of these. */
 enum { LIA_ACT_NONE = 0, LIA_ACT_RELU = 1, LIA_ACT_SILU = 2, LIA_ACT_GELU_ERF = 3, LIA_ACT_GELU_TANH = 4,
-       LIA_ACT_CLAMPED_SWISH = 5 /* gated form only: see lia_moe_gemm_act */ };
+       LIA_ACT_CLAMPED_SWISH = 5 /* gated form only: see lia_moe_gemm_act */,
+       LIA_ACT_RELU_SQUARED = 6 };
 
 /* x[r] = table[ids[r]] as fp32; x_copy (may be NULL) receives the same rows */
 int lia_embed_rows(const int64_t* ids, const void* table, int table_f32, float* x, float* x_copy, int rows, int W, int vocab,
@@ -519,6 +520,46 @@ int lia_moe_gemm_weighted(const void* A, int a_f32, int lda, const void* W, int 
 int lia_moe_combine_gated(const void* ypair, int ypair_f32, const int* pos_of, const float* wt, int weighted, const void* shared, int act_f32,
                           const float* shared_gate, int ldg, const int* idx, int n_real, const void* h, float* y, int M, int W, int top,
                           lia_stream_t stream);
+
+/* ---- Designs that keep several residual streams, run two mixers side by side and recur through a state-space dual or a gated linear
+ * recurrent unit; routers that choose among groups of experts.  (ABI 11) ---- */
+
+/* Residual streams x [rows][S][W] fp32 (S <= 16).  With N(z; w) = w z / sqrt(mean(z^2) + eps):
+ *   v = y, or (w_y given) scale * (N(y; w_y) + N(y2; w_y2)), y2 may be NULL;
+ *   x[t] = sum_s mix[s][t] x[s] + w_out[t] v, all t from the old streams (y NULL: unchanged);
+ *   h = N(sum_s w_in[s] x[s]; w) from the new streams (h NULL: not made). */
+int lia_streams_update(float* x, const void* y, int y_f32, const float* w_y, const void* y2, const float* w_y2, float scale, const float* mix,
+                       const float* w_out, const float* w_in, const float* w, void* h, int h_f32, int rows, int S, int W, float eps,
+                       lia_stream_t stream);
+/* all S streams of row r = table[ids[r]]; h (may be NULL) as above; table and h of the activations' type */
+int lia_streams_embed(const int64_t* ids, const void* table, int act_f32, float* x, const float* w_in, const float* w, void* h, int rows, int S,
+                      int W, int vocab, float eps, lia_stream_t stream);
+/* h[r] = N(sum_s x[rows[r]][s]; w) */
+int lia_streams_gather(const float* x, const int* rows, const float* w, void* h, int h_f32, int n, int S, int W, float eps, lia_stream_t stream);
+/* out[m] = N(o[m] * silu(z[m]); w) with the mean taken over each of `groups` equal parts of the F numbers; z has row stride ldz */
+int lia_silu_gate_norm(const float* o, const void* z, int ldz, const float* w, void* out, int act_f32, int M, int F, int groups, float eps,
+                       lia_stream_t stream);
+/* A short causal convolution (taps <= 16, wconv [C][taps], last column = current token) on the C columns of y from col0 on: the inputs are
+ * y + in_bias (what lies before the sequence's start is zero), out [M][ldo] fp32 = act(sum + bias), act LIA_ACT_NONE or LIA_ACT_SILU;
+ * in_bias and bias may be NULL.  state [slot][taps-1][C] fp32 holds the inputs (without in_bias) before each portion and is moved past
+ * the step's portions.  H > 0: columns dt_col .. dt_col + H - 1 become gates [M][2H] = dt | g with dt = softplus(y + dt_bias[h]),
+ * g = exp(-exp(a_log[h]) dt). */
+int lia_conv_act(const void* y, int y_f32, int ld, int col0, int C, const float* in_bias, const float* wconv, const float* bias, int taps, int act,
+                 float* state, const int* meta, const int* segs, int nseg, float* out, int ldo, int M, int dt_col, int H, const float* dt_bias,
+                 const float* a_log, float* gates, lia_stream_t stream);
+/* State-space dual recurrence over every portion, per head h (B and C of group h / (H / G), N <= 512 numbers; x of vdim numbers; all with
+ * row stride ld):  S = g S + dt B x^T,  o = S^T C + D[h] x;  gates [rows][2H] = dt | g; state_S [slot][H][vdim][N], o [rows][H * vdim] fp32 */
+int lia_ssd_scan(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* state_S, const int* segs, int nseg,
+                 int H, int G, int N, int vdim, float* o, lia_stream_t stream);
+/* Real-gated linear recurrent unit over every portion, channel by channel (width = blocks * n): log a = c sigmoid(r + its bias),
+ * S = a S + sqrt(1 - a^2) sigmoid(i + its bias) u, out = S * gelu_tanh(y + y_bias) of y's type; z [rows][blocks][2n] = r | i,
+ * z_bias [blocks][2n], state [slot][width] fp32; y has row stride ldy, y_bias may be NULL */
+int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
+                   float* state, const int* segs, int nseg, int width, int blocks, void* out, lia_stream_t stream);
+/* lia_router_topk_scored with groups > 1: the experts form that many equal groups of neighbours, a group ranks by its largest choice score
+ * and only experts of the `keep` best groups can be chosen (top <= keep * E / groups) */
+int lia_router_topk_grouped(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int groups, int keep, int* idx,
+                            float* wt, int M, int E, int top, lia_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -19,6 +19,15 @@
 //                      from the rows before it in the same portion, or from the sequence's state), SiLU, q and k made unit
 //                      vectors per head (q also scaled), and the per-head gates beta = sigmoid(.), g = exp(-exp(A) softplus(. + dt)).
 //   conv_state_update: the last taps - 1 inputs of every portion become the sequence's new convolution state.
+//   conv_act:          a short causal convolution over time per channel of ONE column range with an input bias, an output bias and an
+//                      activation, the update of its state, and the step sizes and decays of a state-space recurrence beside it.
+//
+// Two more recurrences, on inputs that conv_act has made fp32:
+//   ssd_scan    (state-space duality, a scalar decay per head and token):   S_t = g_t S_{t-1} + dt_t B_t x_t^T,   y_t = S_t^T C_t + D_h x_t.
+//               State [vdim][N] per (slot, head) as above, but lanes share columns: a thread owns N / 8 rows of two columns, so one 128-bit
+//               read of B or C serves 8 cells and a token's two sums meet in three exchanges.
+//   rglru_scan  (real-gated linear recurrent unit, one number per channel): S_t = a_t S_{t-1} + sqrt(1 - a_t^2) i_t u_t,  out_t = S_t gelu(y_t).
+//               64 tokens at a time: 16 warps fold 4 tokens each into one affine map, the maps are chained through shared memory.
 #include <math.h>
 
 #include "common.cuh"
@@ -417,6 +426,310 @@ int dispatch_scan(const void* q, const void* k, int ldqk, const void* v, int ldv
   return launch_scan<T, 16>(q, k, ldqk, v, ldv, in_silu, decay, gates, St, segs, nseg, H, G, dim, vdim, o, stream);
 }
 
+// ---------------------------------------------------------------------------------------------------- convolution of one column range
+// Thread per channel, walking down a strip of rows with the last taps - 1 inputs in registers.  Input = y[row][col0 + c] + in_bias[c] (zero,
+// without the bias, before the sequence's start); out[row][c] = act(sum_j w[c][taps - 1 - j] * input j tokens back + bias[c]).
+// state [slot][taps-1][C] holds the inputs before their bias.  single: every portion is one row, so the thread that reads a sequence's
+// state is the only one that does and also moves it on.
+// Threads C .. C + H - 1 (H > 0) make the recurrence's per-token numbers instead: gates[row] = dt | g with
+// dt = softplus(y[row][dt_col + h] + dt_bias[h]),  g = exp(-exp(a_log[h]) dt).
+struct ConvActArgs {
+  int ld, col0, C, taps, act, single, ldo, M, strip;
+  int dt_col, H;
+};
+
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z))); }
+
+template <typename T, int TM>
+__global__ void __launch_bounds__(256) conv_act_kernel(const T* __restrict__ y, const float* __restrict__ in_bias, const float* __restrict__ wconv,
+                                                       const float* __restrict__ bias, float* __restrict__ state, const int* __restrict__ meta,
+                                                       float* __restrict__ out, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                                                       float* __restrict__ gates, ConvActArgs a) {
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  const int r0 = blockIdx.y * a.strip, r1 = min(a.M, r0 + a.strip);
+  if (c >= a.C + a.H) return;
+  if (c >= a.C) {
+    const int h = c - a.C;
+    const float rate = -expf(a_log[h]), b = dt_bias[h];
+    for (int r = r0; r < r1; ++r) {
+      const float z = ldf(y + (size_t)r * a.ld + a.dt_col + h) + b;
+      const float dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+      gates[(size_t)r * 2 * a.H + h] = dt;
+      gates[(size_t)r * 2 * a.H + a.H + h] = expf(rate * dt);
+    }
+    return;
+  }
+  const T* col = y + a.col0 + c;
+  const float ib = in_bias ? in_bias[c] : 0.f, ob = bias ? bias[c] : 0.f;
+  float w[TM], win[TM];                          // by tokens back
+#pragma unroll
+  for (int j = 0; j < TM; ++j) {
+    w[j] = j < a.taps ? wconv[(size_t)c * a.taps + a.taps - 1 - j] : 0.f;
+    win[j] = 0.f;
+  }
+  int pslot = -1, ppos = -1;
+  for (int r = r0; r < r1; ++r) {
+    const int slot = meta[2 * r], pos = meta[2 * r + 1];
+    float* st = state ? state + (size_t)slot * (a.taps - 1) * a.C + c : nullptr;
+    if (r > r0 && slot == pslot && pos == ppos + 1) {
+#pragma unroll
+      for (int j = TM - 1; j > 0; --j) win[j] = win[j - 1];
+    } else {
+      int inside = 1;                            // rows r-1 .. r-(inside-1) belong to this portion
+      while (inside < a.taps && r - inside >= 0 && meta[2 * (r - inside)] == slot && meta[2 * (r - inside) + 1] == pos - inside) ++inside;
+#pragma unroll
+      for (int j = 1; j < TM; ++j) {
+        win[j] = 0.f;
+        if (j < a.taps && j <= pos)
+          win[j] = j < inside ? ldf(col + (size_t)(r - j) * a.ld) : st[(size_t)(inside - 1 - j + a.taps - 1) * a.C];
+      }
+    }
+    win[0] = ldf(col + (size_t)r * a.ld);
+    float acc = 0.f;
+#pragma unroll
+    for (int j = 0; j < TM; ++j)
+      if (j < a.taps && j <= pos) acc = fmaf(w[j], win[j] + ib, acc);
+    acc += ob;
+    if (a.act == LIA_ACT_SILU) acc = silu(acc);
+    out[(size_t)r * a.ldo + c] = acc;
+    if (a.single) {
+#pragma unroll
+      for (int j = 0; j < TM - 1; ++j)
+        if (j < a.taps - 1) st[(size_t)(a.taps - 2 - j) * a.C] = win[j];
+    }
+    pslot = slot;
+    ppos = pos;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------- state-space duality
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+constexpr int SSD_TB = 8;         // tokens per stage
+constexpr int SSD_COLS = 32;      // columns (of vdim) per block: 4 warps x 8
+
+// Block: 32 columns of one head of one portion.  Lane: row group rg = lane & 7 owns rows 32 j + 4 rg .. + 3 (j < NJ, N <= 32 NJ), column
+// group lane >> 3 owns two columns.  Stages of SSD_TB tokens (B | C | x of this block's columns | dt | g) arrive by cp.async one stage ahead.
+template <int NJ, bool VL>
+__global__ void __launch_bounds__(128) ssd_scan_kernel(const float* __restrict__ B, const float* __restrict__ C, const float* __restrict__ x, int ld,
+                                                       const float* __restrict__ gates, const float* __restrict__ D, float* __restrict__ St,
+                                                       const int* __restrict__ segs, int H, int G, int N, int vdim, float* __restrict__ o) {
+  constexpr int NP = NJ * 32, ROWF = 2 * NP + SSD_COLS + 4;
+  extern __shared__ __align__(16) float stage[];       // [2][SSD_TB][ROWF]
+  const int seg = blockIdx.z, h = blockIdx.y, colb = blockIdx.x * SSD_COLS, g = h / (H / G);
+  const int slot = segs[4 * seg], row0 = segs[4 * seg + 2], len = segs[4 * seg + 3];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7;
+  const int cl = warp * 8 + (lane >> 3) * 2, col0 = colb + cl;
+  const int ncol = min(SSD_COLS, vdim - colb);
+
+  for (int i = threadIdx.x; i < 2 * SSD_TB * ROWF; i += 128) stage[i] = 0.f;      // rows N .. NP-1 of B and C stay zero
+  float S[2][NJ * 4];
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    const float* Sp = St + (((size_t)slot * H + h) * vdim + col0 + c) * N;
+    const bool live = col0 + c < vdim;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int r = 32 * j + 4 * rg;
+      if (VL) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (live && r < N) v = *reinterpret_cast<const float4*>(Sp + r);
+        S[c][4 * j] = v.x; S[c][4 * j + 1] = v.y; S[c][4 * j + 2] = v.z; S[c][4 * j + 3] = v.w;
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[c][4 * j + e] = (live && r + e < N) ? Sp[r + e] : 0.f;
+      }
+    }
+  }
+  __syncthreads();
+
+  constexpr int U = VL ? 4 : 1;                        // floats per copy
+  const int n_u = N / U, x_u = VL ? ncol / 4 : ncol, per_tok = 2 * n_u + x_u;
+  auto fetch = [&](int gidx) {
+    const int t0 = gidx * SSD_TB, nt = min(SSD_TB, len - t0);
+    float* st = stage + (gidx & 1) * SSD_TB * ROWF;
+    for (int e = threadIdx.x; e < nt * per_tok; e += 128) {
+      const int t = e / per_tok, j = e - t * per_tok;
+      const size_t row = (size_t)(row0 + t0 + t) * ld;
+      const float* src;
+      float* dst = st + t * ROWF;
+      if (j < n_u) { src = B + row + g * N + j * U; dst += j * U; }
+      else if (j < 2 * n_u) { src = C + row + g * N + (j - n_u) * U; dst += NP + (j - n_u) * U; }
+      else { src = x + row + (size_t)h * vdim + colb + (j - 2 * n_u) * U; dst += 2 * NP + (j - 2 * n_u) * U; }
+      if (VL) cp_async16(dst, src);
+      else cp_async4(dst, src);
+    }
+    if (threadIdx.x < 2 * nt) {
+      const int t = threadIdx.x >> 1, which = threadIdx.x & 1;
+      cp_async4(st + t * ROWF + 2 * NP + SSD_COLS + which, gates + (size_t)(row0 + t0 + t) * 2 * H + which * H + h);
+    }
+  };
+  const float dh = D[h];
+  const int groups = (len + SSD_TB - 1) / SSD_TB;
+  fetch(0);
+  cp_async_commit();
+  for (int gi = 0; gi < groups; ++gi) {
+    if (gi + 1 < groups) fetch(gi + 1);
+    cp_async_commit();
+    cp_async_wait<1>();
+    __syncthreads();
+    const float* st = stage + (gi & 1) * SSD_TB * ROWF;
+    const int nt = min(SSD_TB, len - gi * SSD_TB);
+    float* orow = o + (size_t)(row0 + gi * SSD_TB) * H * vdim + (size_t)h * vdim + colb;
+#pragma unroll 2
+    for (int t = 0; t < nt; ++t) {
+      const float* tk = st + t * ROWF;
+      const float2 xv = *reinterpret_cast<const float2*>(tk + 2 * NP + cl);
+      const float2 dg = *reinterpret_cast<const float2*>(tk + 2 * NP + SSD_COLS);
+      const float u0 = dg.x * xv.x, u1 = dg.x * xv.y;
+      float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const float4 k = *reinterpret_cast<const float4*>(tk + 32 * j + 4 * rg);
+        const float4 q = *reinterpret_cast<const float4*>(tk + NP + 32 * j + 4 * rg);
+        S[0][4 * j] = fmaf(dg.y, S[0][4 * j], k.x * u0);
+        S[1][4 * j] = fmaf(dg.y, S[1][4 * j], k.x * u1);
+        a0 = fmaf(S[0][4 * j], q.x, a0);
+        a1 = fmaf(S[1][4 * j], q.x, a1);
+        S[0][4 * j + 1] = fmaf(dg.y, S[0][4 * j + 1], k.y * u0);
+        S[1][4 * j + 1] = fmaf(dg.y, S[1][4 * j + 1], k.y * u1);
+        b0 = fmaf(S[0][4 * j + 1], q.y, b0);
+        b1 = fmaf(S[1][4 * j + 1], q.y, b1);
+        S[0][4 * j + 2] = fmaf(dg.y, S[0][4 * j + 2], k.z * u0);
+        S[1][4 * j + 2] = fmaf(dg.y, S[1][4 * j + 2], k.z * u1);
+        a0 = fmaf(S[0][4 * j + 2], q.z, a0);
+        a1 = fmaf(S[1][4 * j + 2], q.z, a1);
+        S[0][4 * j + 3] = fmaf(dg.y, S[0][4 * j + 3], k.w * u0);
+        S[1][4 * j + 3] = fmaf(dg.y, S[1][4 * j + 3], k.w * u1);
+        b0 = fmaf(S[0][4 * j + 3], q.w, b0);
+        b1 = fmaf(S[1][4 * j + 3], q.w, b1);
+      }
+      a0 += b0;
+      a1 += b1;
+      // even row groups go on with column 0, odd ones with column 1
+      const bool odd = rg & 1;
+      float sum = (odd ? a1 : a0) + __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+      if (rg < 2 && cl + rg < ncol) orow[(size_t)t * H * vdim + cl + rg] = fmaf(dh, odd ? xv.y : xv.x, sum);
+    }
+    __syncthreads();                                   // the stage after next goes where this one was
+  }
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    if (col0 + c >= vdim) continue;
+    float* Sp = St + (((size_t)slot * H + h) * vdim + col0 + c) * N;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int r = 32 * j + 4 * rg;
+      if (VL) {
+        if (r < N) *reinterpret_cast<float4*>(Sp + r) = make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (r + e < N) Sp[r + e] = S[c][4 * j + e];
+      }
+    }
+  }
+}
+
+template <int NJ, bool VL>
+int launch_ssd_as(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs, int nseg, int H,
+                  int G, int N, int vdim, float* o, cudaStream_t stream) {
+  const size_t smem = (size_t)2 * SSD_TB * (2 * NJ * 32 + SSD_COLS + 4) * sizeof(float);
+  if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(ssd_scan_kernel<NJ, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  dim3 grid((vdim + SSD_COLS - 1) / SSD_COLS, H, nseg);
+  ssd_scan_kernel<NJ, VL><<<grid, 128, smem, stream>>>(B, C, x, ld, gates, D, St, segs, H, G, N, vdim, o);
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
+}
+
+// 128-bit copies and state accesses: every B, C, x segment and every state column starts on a 16-byte boundary
+template <int NJ>
+int launch_ssd(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs, int nseg, int H,
+               int G, int N, int vdim, float* o, cudaStream_t stream) {
+  const bool aligned = ((reinterpret_cast<uintptr_t>(B) | reinterpret_cast<uintptr_t>(C) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(St)) % 16 == 0) &&
+                       ld % 4 == 0 && N % 4 == 0 && vdim % 4 == 0;
+  if (aligned) return launch_ssd_as<NJ, true>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
+  return launch_ssd_as<NJ, false>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
+}
+
+// ---------------------------------------------------------------------------------------------------- gated linear recurrent unit
+constexpr int LRU_W = 16, LRU_T = 4;          // warps per block, tokens per warp and sweep
+
+// Block: 32 channels of one portion.  z [rows][blocks][2 n] holds every channel block's gate projections r | i (n = width / blocks),
+// z_bias [blocks][2 n] their biases, c[ch] = -8 softplus(lam): log a = c sigmoid(r).
+template <typename T>
+__global__ void __launch_bounds__(LRU_W * 32) rglru_scan_kernel(const float* __restrict__ u, const float* __restrict__ z, const float* __restrict__ z_bias,
+                                                                const float* __restrict__ c, const T* __restrict__ y, int ldy, const float* __restrict__ y_bias,
+                                                                float* __restrict__ St, const int* __restrict__ segs, int width, int n, T* __restrict__ out) {
+  __shared__ float2 maps[2][LRU_W][32];       // a warp's four tokens as S -> x S + y
+  const int seg = blockIdx.y, slot = segs[4 * seg], row0 = segs[4 * seg + 2], len = segs[4 * seg + 3];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ch = blockIdx.x * 32 + lane;
+  const bool live = ch < width;
+  const int blk = live ? ch / n : 0, zc = blk * 2 * n + (live ? ch - blk * n : 0);
+  const float cc = live ? c[ch] : 0.f, rb = live ? z_bias[zc] : 0.f, ib = live ? z_bias[zc + n] : 0.f, yb = (live && y_bias) ? y_bias[ch] : 0.f;
+  float S = live ? St[(size_t)slot * width + ch] : 0.f;
+  float ur[LRU_T], zr[LRU_T], zi[LRU_T], yr[LRU_T];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) {
+      const int t = t0 + warp * LRU_T + k;
+      ur[k] = zr[k] = zi[k] = yr[k] = 0.f;
+      if (live && t < len) {
+        const size_t row = (size_t)(row0 + t);
+        ur[k] = u[row * width + ch];
+        zr[k] = z[row * 2 * width + zc];
+        zi[k] = z[row * 2 * width + zc + n];
+        yr[k] = ldf(y + row * ldy + ch);
+      }
+    }
+  };
+  fetch(0);
+  int buf = 0;
+  for (int t0 = 0; t0 < len; t0 += LRU_W * LRU_T) {
+    float a[LRU_T], b[LRU_T], g[LRU_T], pa = 1.f, pb = 0.f;
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) {
+      a[k] = 1.f;
+      b[k] = g[k] = 0.f;
+      if (t0 + warp * LRU_T + k < len) {
+        const float la = cc / (1.0f + expf(-(zr[k] + rb)));
+        a[k] = expf(la);
+        b[k] = sqrtf(-expm1f(2.0f * la)) * ur[k] / (1.0f + expf(-(zi[k] + ib)));
+        g[k] = gelu_tanh(yr[k] + yb);
+      }
+      pa *= a[k];
+      pb = fmaf(a[k], pb, b[k]);
+    }
+    maps[buf][warp][lane] = make_float2(pa, pb);
+    if (t0 + LRU_W * LRU_T < len) fetch(t0 + LRU_W * LRU_T);
+    __syncthreads();
+    float s = S;
+#pragma unroll
+    for (int w = 0; w < LRU_W; ++w) {
+      if (w == warp) s = S;
+      const float2 m = maps[buf][w][lane];
+      S = fmaf(m.x, S, m.y);
+    }
+#pragma unroll
+    for (int k = 0; k < LRU_T; ++k) {
+      const int t = t0 + warp * LRU_T + k;
+      s = fmaf(a[k], s, b[k]);
+      if (live && t < len) out[(size_t)(row0 + t) * width + ch] = T(s * g[k]);
+    }
+    buf ^= 1;                                 // the other half: last read before the barrier above
+  }
+  if (warp == 0 && live) St[(size_t)slot * width + ch] = S;
+}
+
 }  // namespace
 
 extern "C" int lia_conv_prep(const void* y, int y_f32, int ld, int q_off, int k_off, int v_off, const float* wconv, const float* conv_state,
@@ -486,4 +799,62 @@ extern "C" int lia_forget_scan(const float* q, const float* f, int ldqf, const f
   LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && H > 0 && H <= 65535 && dim > 0 && dim <= 512 && vdim > 0,
                 "lia_forget_scan: bad shape nseg=%d H=%d dim=%d vdim=%d", nseg, H, dim, vdim);
   return dispatch_scan<float>(q, f, ldqf, v, ldv, 0, nullptr, nullptr, state_S, segs, nseg, H, H, dim, vdim, o, stream);
+}
+
+/* see lia_b200.h */
+extern "C" int lia_conv_act(const void* y, int y_f32, int ld, int col0, int C, const float* in_bias, const float* wconv, const float* bias, int taps,
+                            int act, float* state, const int* meta, const int* segs, int nseg, float* out, int ldo, int M, int dt_col, int H,
+                            const float* dt_bias, const float* a_log, float* gates, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(y && wconv && meta && segs && out && M > 0 && C > 0 && nseg > 0 && nseg <= 65535 && nseg <= M, "lia_conv_act: bad arguments");
+  LIA_CHECK_ARG(taps >= 1 && taps <= MAX_TAPS && (taps == 1 || state) && ldo >= C && ld >= col0 + C && col0 >= 0, "lia_conv_act: bad shape C=%d taps=%d", C, taps);
+  LIA_CHECK_ARG(act == LIA_ACT_NONE || act == LIA_ACT_SILU, "lia_conv_act: unknown activation %d", act);
+  LIA_CHECK_ARG(H >= 0 && (H == 0 || (dt_bias && a_log && gates && dt_col >= 0 && ld >= dt_col + H)), "lia_conv_act: bad step sizes (H=%d)", H);
+  const int single = nseg == M && taps > 1;      // every portion is one row
+  ConvActArgs a{ld, col0, C, taps, act, single, ldo, M, M <= 64 ? 1 : 8, dt_col, H};
+  dim3 grid((C + H + 255) / 256, (M + a.strip - 1) / a.strip);
+  LIA_CHECK_ARG(grid.y <= 65535, "lia_conv_act: too many rows (%d)", M);
+#define LIA_CA(T, TM) conv_act_kernel<T, TM><<<grid, 256, 0, stream>>>(reinterpret_cast<const T*>(y), in_bias, wconv, bias, state, meta, out, dt_bias, a_log, gates, a)
+  if (y_f32) {
+    if (taps <= 4) LIA_CA(float, 4);
+    else LIA_CA(float, MAX_TAPS);
+  } else {
+    if (taps <= 4) LIA_CA(bf16, 4);
+    else LIA_CA(bf16, MAX_TAPS);
+  }
+#undef LIA_CA
+  LIA_LAUNCH_CHECK();
+  if (taps > 1 && !single) {
+    ConvCols cc{col0, 0, 0, C, 0, 0};
+    dim3 g2((C + 255) / 256, nseg);
+    if (y_f32) conv_state_update_kernel<float><<<g2, 256, 0, stream>>>(reinterpret_cast<const float*>(y), ld, cc, state, segs, taps);
+    else conv_state_update_kernel<bf16><<<g2, 256, 0, stream>>>(reinterpret_cast<const bf16*>(y), ld, cc, state, segs, taps);
+    LIA_LAUNCH_CHECK();
+  }
+  return LIA_OK;
+}
+
+extern "C" int lia_ssd_scan(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* state_S, const int* segs,
+                            int nseg, int H, int G, int N, int vdim, float* o, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(B && C && x && gates && D && state_S && segs && o, "lia_ssd_scan: null pointer");
+  LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && N > 0 && N <= 512 && vdim > 0,
+                "lia_ssd_scan: bad shape nseg=%d H=%d G=%d N=%d vdim=%d", nseg, H, G, N, vdim);
+  if (N <= 32) return launch_ssd<1>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 64) return launch_ssd<2>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 128) return launch_ssd<4>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 256) return launch_ssd<8>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  return launch_ssd<16>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+}
+
+extern "C" int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
+                              float* state, const int* segs, int nseg, int width, int blocks, void* out, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(u && z && z_bias && c && y && state && segs && out, "lia_rglru_scan: null pointer");
+  LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && width > 0 && blocks > 0 && width % blocks == 0 && ldy >= width, "lia_rglru_scan: bad shape width=%d blocks=%d", width, blocks);
+  dim3 grid((width + 31) / 32, nseg);
+  if (y_f32) rglru_scan_kernel<float><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const float*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<float*>(out));
+  else rglru_scan_kernel<bf16><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const bf16*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<bf16*>(out));
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
 }

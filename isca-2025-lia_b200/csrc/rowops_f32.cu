@@ -1,6 +1,7 @@
 // Row operations of models that keep their residual stream in 32-bit floats: RMS norms with a scalar or a per-channel
 // weight (fused with the residual add that follows a sublayer and with the norm that precedes the next one), the token
 // embedding with its norm, with learned or wave positions and with a bigram table, the gated, normed residual update with a weighted mix of all earlier layers' results, the
+// residual kept as several streams that learned weights read, mix and write, a gate product behind a norm in groups, the
 // polynomial activation between norms, a gated feed-forward activation with clamps, a projection onto a handful of outputs with the
 // gate non-linearities in its epilogue, a plain strided-batched projection on the CUDA cores (true 32-bit products and
 // sums: the exact path, and the carrier of shapes the tensor-core GEMM does not take), and a 32-bit argmax.
@@ -265,6 +266,215 @@ __global__ void __launch_bounds__(256) gated_rms_add_kernel(float* __restrict__ 
     }
     if (y != nullptr || stack != nullptr) x[base + i] = v;
     if (h != nullptr) stf(h + base + i, v);
+  }
+}
+
+// VEC (4 or 1) consecutive numbers of a row as floats, and back
+template <int VEC> __device__ __forceinline__ void ld_vec(const float* p, float* f) {
+  if constexpr (VEC == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int VEC> __device__ __forceinline__ void ld_vec(const bf16* p, float* f) {
+  if constexpr (VEC == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    unpack_bf16x2(v.x, f[0], f[1]);
+    unpack_bf16x2(v.y, f[2], f[3]);
+  } else {
+    f[0] = __bfloat162float(*p);
+  }
+}
+template <int VEC> __device__ __forceinline__ void st_vec(float* p, const float* f) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int VEC> __device__ __forceinline__ void st_vec(bf16* p, const float* f) {
+  if constexpr (VEC == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+  else *p = __float2bfloat16_rn(f[0]);
+}
+
+// Designs that keep S residual streams per token, x [rows][S][W] fp32, instead of one:
+//   v      = y                                                   (w_y null)
+//            scale * (N(y; w_y) + N(y2; w_y2))                   (two branches side by side; y2 may be null)
+//   x[t]   = sum_s mix[s][t] x[s] + w_out[t] v                   (all t from the old streams; y null: the streams stay as they are)
+//   h      = N(sum_s w_in[s] x[s]; w)                            (what the next sublayer reads; h null: not made)
+// N(z; w) = w z / sqrt(mean(z^2) + eps).  ids given: the streams start as S copies of table[ids[row]] (y is null then).
+// Block per row, SM >= S streams in registers; `us` (dynamic shared memory, W floats) keeps the read-out for its norm.
+template <typename TY, typename TH, int SM, int VEC>
+__global__ void __launch_bounds__(256) streams_kernel(float* __restrict__ x, const TY* __restrict__ y, const float* __restrict__ w_y, const TY* __restrict__ y2,
+                                                      const float* __restrict__ w_y2, float scale, const float* __restrict__ mix,
+                                                      const float* __restrict__ w_out, const float* __restrict__ w_in, const float* __restrict__ w,
+                                                      TH* __restrict__ h, const int64_t* __restrict__ ids, const TH* __restrict__ table, int vocab, int S,
+                                                      int W, float eps) {
+  extern __shared__ __align__(16) float us[];
+  __shared__ float red[8];
+  __shared__ float cmix[SM * SM], cout[SM], cin[SM];
+  const size_t row = blockIdx.x;
+  float* xr = x + row * S * W;
+  for (int i = threadIdx.x; i < S * S; i += 256) cmix[(i / S) * SM + i % S] = y ? mix[i] : 0.f;
+  for (int i = threadIdx.x; i < S; i += 256) {
+    cout[i] = y ? w_out[i] : 0.f;
+    cin[i] = h ? w_in[i] : 0.f;
+  }
+  const TY* yr = y ? y + row * W : nullptr;
+  const TY* y2r = y2 ? y2 + row * W : nullptr;
+  float n1 = 1.f, n2 = 0.f;
+  if (w_y != nullptr) {
+    float s1 = 0.f, s2 = 0.f;
+    for (int i = threadIdx.x * VEC; i < W; i += 256 * VEC) {
+      float f[VEC];
+      ld_vec<VEC>(yr + i, f);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s1 += f[e] * f[e];
+      if (y2r) {
+        ld_vec<VEC>(y2r + i, f);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s2 += f[e] * f[e];
+      }
+    }
+    n1 = scale / sqrtf(block_sum<256>(s1, red) / (float)W + eps);
+    if (y2r) n2 = scale / sqrtf(block_sum<256>(s2, red) / (float)W + eps);
+  }
+  __syncthreads();
+  const TH* er = nullptr;
+  if (ids != nullptr) {
+    long long id = ids[row];
+    if (id < 0 || id >= vocab) id = 0;     // the host checks the range; never read outside the table
+    er = table + (size_t)id * W;
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x * VEC; i < W; i += 256 * VEC) {
+    float xv[SM][VEC], u[VEC];
+    if (er != nullptr) {
+      float f[VEC];
+      ld_vec<VEC>(er + i, f);
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) xv[s][e] = f[e];
+          st_vec<VEC>(xr + (size_t)s * W + i, f);
+        }
+    } else {
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) ld_vec<VEC>(xr + (size_t)s * W + i, xv[s]);
+    }
+    if (yr != nullptr) {
+      float v[VEC];
+      ld_vec<VEC>(yr + i, v);
+      if (w_y != nullptr) {
+        float wv[VEC];
+        ld_vec<VEC>(w_y + i, wv);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] *= n1 * wv[e];
+        if (y2r) {
+          float f[VEC];
+          ld_vec<VEC>(y2r + i, f);
+          ld_vec<VEC>(w_y2 + i, wv);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[e] = fmaf(f[e] * n2, wv[e], v[e]);
+        }
+      }
+      float nx[SM][VEC];
+#pragma unroll
+      for (int t = 0; t < SM; ++t)
+        if (t < S) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) nx[t][e] = cout[t] * v[e];
+#pragma unroll
+          for (int s = 0; s < SM; ++s)
+            if (s < S) {
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) nx[t][e] = fmaf(cmix[s * SM + t], xv[s][e], nx[t][e]);
+            }
+          st_vec<VEC>(xr + (size_t)t * W + i, nx[t]);
+        }
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) xv[s][e] = nx[s][e];
+        }
+    }
+    if (h != nullptr) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) u[e] = 0.f;
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) u[e] = fmaf(cin[s], xv[s][e], u[e]);
+        }
+      st_vec<VEC>(us + i, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += u[e] * u[e];
+    }
+  }
+  if (h == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum<256>(ss, red) / (float)W + eps);
+  for (int i = threadIdx.x * VEC; i < W; i += 256 * VEC) {          // each thread re-reads only what it wrote
+    float u[VEC], wv[VEC];
+    ld_vec<VEC>(us + i, u);
+    ld_vec<VEC>(w + i, wv);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u[e] *= inv * wv[e];
+    st_vec<VEC>(h + row * W + i, u);
+  }
+}
+
+// h[r] = N(sum_s x[rows[r]][s]; w): the norm of a few selected rows of a residual kept as S streams
+template <typename TH>
+__global__ void __launch_bounds__(256) streams_gather_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ w,
+                                                             TH* __restrict__ h, int S, int W, float eps) {
+  extern __shared__ __align__(16) float us[];
+  __shared__ float red[8];
+  const float* xr = x + (size_t)rows[blockIdx.x] * S * W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    float u = 0.f;
+    for (int s = 0; s < S; ++s) u += xr[(size_t)s * W + i];
+    us[i] = u;
+    ss += u * u;
+  }
+  const float inv = 1.0f / sqrtf(block_sum<256>(ss, red) / (float)W + eps);
+  for (int i = threadIdx.x; i < W; i += 256) stf(h + (size_t)blockIdx.x * W + i, us[i] * inv * w[i]);
+}
+
+// out = w * g / sqrt(mean(g^2) + eps), g = o * silu(z), the mean taken over each of `groups` equal parts of a row by itself (the gate comes
+// before the norm).  o fp32 [M][F], z of the activations' type with row stride ldz.  Block per (row, part); `us` keeps g (F / groups floats).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) silu_gate_norm_kernel(const float* __restrict__ o, const T* __restrict__ z, int ldz, const float* __restrict__ w,
+                                                             T* __restrict__ out, int F, int groups, float eps) {
+  extern __shared__ __align__(16) float us[];
+  __shared__ float red[4];
+  const size_t row = blockIdx.x / groups;
+  const int n = F / groups, first = (int)(blockIdx.x % groups) * n;
+  const float* orow = o + row * F + first;
+  const T* zrow = z + row * ldz + first;
+  float ss = 0.f;
+  for (int i = threadIdx.x * VEC; i < n; i += 128 * VEC) {
+    float ov[VEC], zv[VEC];
+    ld_vec<VEC>(orow + i, ov);
+    ld_vec<VEC>(zrow + i, zv);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      ov[e] *= zv[e] / (1.0f + expf(-zv[e]));
+      ss += ov[e] * ov[e];
+    }
+    st_vec<VEC>(us + i, ov);
+  }
+  const float inv = 1.0f / sqrtf(block_sum<128>(ss, red) / (float)n + eps);
+  for (int i = threadIdx.x * VEC; i < n; i += 128 * VEC) {
+    float g[VEC], wv[VEC];
+    ld_vec<VEC>(us + i, g);
+    ld_vec<VEC>(w + first + i, wv);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) g[e] *= inv * wv[e];
+    st_vec<VEC>(out + row * F + first + i, g);
   }
 }
 
@@ -764,6 +974,103 @@ extern "C" int lia_embed_bigram_pos(const int64_t* ids, const void* table, const
   else if (h_f32) LIA_EBP(bf16, float);
   else LIA_EBP(bf16, bf16);
 #undef LIA_EBP
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
+}
+
+namespace {
+
+template <typename TY, typename TH, int SM, int VEC>
+int launch_streams(float* x, const void* y, const float* w_y, const void* y2, const float* w_y2, float scale, const float* mix, const float* w_out,
+                   const float* w_in, const float* w, void* h, const int64_t* ids, const void* table, int vocab, int rows, int S, int W, float eps,
+                   cudaStream_t stream) {
+  const size_t smem = h ? (size_t)W * sizeof(float) : 0;
+  if (smem > 40 * 1024) LIA_CUDA(cudaFuncSetAttribute(streams_kernel<TY, TH, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  streams_kernel<TY, TH, SM, VEC><<<rows, 256, smem, stream>>>(x, reinterpret_cast<const TY*>(y), w_y, reinterpret_cast<const TY*>(y2), w_y2, scale, mix, w_out,
+                                                               w_in, w, reinterpret_cast<TH*>(h), ids, reinterpret_cast<const TH*>(table), vocab, S, W, eps);
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
+}
+
+template <typename TY, typename TH, int VEC, typename... A>
+int dispatch_streams_n(int S, A... args) {
+  if (S <= 2) return launch_streams<TY, TH, 2, VEC>(args...);
+  if (S <= 4) return launch_streams<TY, TH, 4, VEC>(args...);
+  if (S <= 8) return launch_streams<TY, TH, 8, VEC>(args...);
+  return launch_streams<TY, TH, 16, 1>(args...);
+}
+
+bool vec4_ok(const void* p, size_t elem) { return reinterpret_cast<uintptr_t>(p) % (4 * elem) == 0; }
+
+template <typename TY, typename TH>
+int dispatch_streams(float* x, const void* y, const float* w_y, const void* y2, const float* w_y2, float scale, const float* mix, const float* w_out,
+                     const float* w_in, const float* w, void* h, const int64_t* ids, const void* table, int vocab, int rows, int S, int W, float eps,
+                     cudaStream_t stream) {
+  const bool vec = W % 4 == 0 && vec4_ok(x, 4) && vec4_ok(y, sizeof(TY)) && vec4_ok(y2, sizeof(TY)) && vec4_ok(w_y, 4) && vec4_ok(w_y2, 4) && vec4_ok(w, 4) &&
+                   vec4_ok(h, sizeof(TH)) && vec4_ok(table, sizeof(TH));
+  if (vec) return dispatch_streams_n<TY, TH, 4>(S, x, y, w_y, y2, w_y2, scale, mix, w_out, w_in, w, h, ids, table, vocab, rows, S, W, eps, stream);
+  return dispatch_streams_n<TY, TH, 1>(S, x, y, w_y, y2, w_y2, scale, mix, w_out, w_in, w, h, ids, table, vocab, rows, S, W, eps, stream);
+}
+
+}  // namespace
+
+extern "C" int lia_streams_update(float* x, const void* y, int y_f32, const float* w_y, const void* y2, const float* w_y2, float scale, const float* mix,
+                                  const float* w_out, const float* w_in, const float* w, void* h, int h_f32, int rows, int S, int W, float eps,
+                                  lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(x && (y || h) && (!y || (mix && w_out)) && (!h || (w_in && w)), "lia_streams_update: bad arguments");
+  LIA_CHECK_ARG((!w_y || y) && (!y2 || (w_y && w_y2)), "lia_streams_update: branches and their norms go together");
+  LIA_CHECK_ARG(rows > 0 && S > 0 && S <= 16 && W > 0 && (size_t)W * 4 <= 160 * 1024, "lia_streams_update: bad shape rows=%d S=%d W=%d", rows, S, W);
+#define LIA_SU(TY, TH) return dispatch_streams<TY, TH>(x, y, w_y, y2, w_y2, scale, mix, w_out, w_in, w, h, nullptr, nullptr, 0, rows, S, W, eps, stream)
+  if (y_f32 && h_f32) LIA_SU(float, float);
+  if (y_f32) LIA_SU(float, bf16);
+  if (h_f32) LIA_SU(bf16, float);
+  LIA_SU(bf16, bf16);
+#undef LIA_SU
+}
+
+extern "C" int lia_streams_embed(const int64_t* ids, const void* table, int act_f32, float* x, const float* w_in, const float* w, void* h, int rows, int S,
+                                 int W, int vocab, float eps, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(ids && table && x && vocab > 0 && (!h || (w_in && w)), "lia_streams_embed: bad arguments");
+  LIA_CHECK_ARG(rows > 0 && S > 0 && S <= 16 && W > 0 && (size_t)W * 4 <= 160 * 1024, "lia_streams_embed: bad shape rows=%d S=%d W=%d", rows, S, W);
+  if (act_f32) return dispatch_streams<float, float>(x, nullptr, nullptr, nullptr, nullptr, 1.f, nullptr, nullptr, w_in, w, h, ids, table, vocab, rows, S, W, eps, stream);
+  return dispatch_streams<bf16, bf16>(x, nullptr, nullptr, nullptr, nullptr, 1.f, nullptr, nullptr, w_in, w, h, ids, table, vocab, rows, S, W, eps, stream);
+}
+
+extern "C" int lia_streams_gather(const float* x, const int* rows, const float* w, void* h, int h_f32, int n, int S, int W, float eps, lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(x && rows && w && h && n > 0 && S > 0 && W > 0 && (size_t)W * 4 <= 160 * 1024, "lia_streams_gather: bad arguments");
+  const size_t smem = (size_t)W * sizeof(float);
+  if (h_f32) {
+    if (smem > 40 * 1024) LIA_CUDA(cudaFuncSetAttribute(streams_gather_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    streams_gather_kernel<float><<<n, 256, smem, stream>>>(x, rows, w, reinterpret_cast<float*>(h), S, W, eps);
+  } else {
+    if (smem > 40 * 1024) LIA_CUDA(cudaFuncSetAttribute(streams_gather_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    streams_gather_kernel<bf16><<<n, 256, smem, stream>>>(x, rows, w, reinterpret_cast<bf16*>(h), S, W, eps);
+  }
+  LIA_LAUNCH_CHECK();
+  return LIA_OK;
+}
+
+extern "C" int lia_silu_gate_norm(const float* o, const void* z, int ldz, const float* w, void* out, int act_f32, int M, int F, int groups, float eps,
+                                  lia_stream_t stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  LIA_CHECK_ARG(o && z && w && out && M > 0 && F > 0 && groups > 0 && F % groups == 0 && ldz >= F, "lia_silu_gate_norm: bad arguments (F=%d groups=%d)", F, groups);
+  LIA_CHECK_ARG((size_t)(F / groups) * 4 <= 160 * 1024 && (long long)M * groups <= 0x7fffffff, "lia_silu_gate_norm: bad shape M=%d F=%d groups=%d", M, F, groups);
+  const size_t smem = (size_t)(F / groups) * sizeof(float), elem = act_f32 ? 4 : 2;
+  const bool vec = (F / groups) % 4 == 0 && ldz % 4 == 0 && vec4_ok(o, 4) && vec4_ok(z, elem) && vec4_ok(w, 4) && vec4_ok(out, elem);
+  const unsigned grid = (unsigned)((long long)M * groups);
+#define LIA_SGN(T, VEC)                                                                                                      \
+  do {                                                                                                                       \
+    if (smem > 40 * 1024) LIA_CUDA(cudaFuncSetAttribute(silu_gate_norm_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    silu_gate_norm_kernel<T, VEC><<<grid, 128, smem, stream>>>(o, reinterpret_cast<const T*>(z), ldz, w, reinterpret_cast<T*>(out), F, groups, eps); \
+  } while (0)
+  if (act_f32 && vec) LIA_SGN(float, 4);
+  else if (act_f32) LIA_SGN(float, 1);
+  else if (vec) LIA_SGN(bf16, 4);
+  else LIA_SGN(bf16, 1);
+#undef LIA_SGN
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }

@@ -4,7 +4,8 @@
 //   ln_add_norm    x += mult * LN_post(y);  x += extra;  h = LN_pre(x)    (each part optional, one pass over the row)
 //   ln_gather      h[r] = LN(x[rows[r]]) for the few rows whose logits are wanted
 //   gated_act      out = act(gate) * up  (or act(gate) alone) on column ranges of one projection's output
-//   router_topk    softmax over the experts' logits or a sigmoid of each, the `top` largest (by score, or by score plus a correction), renormalised or not
+//   router_topk    softmax over the experts' logits or a sigmoid of each, the `top` largest (by score, or by score plus a correction), renormalised or not,
+//                  among all experts or those of the best groups
 //   moe_plan       (token, choice) pairs grouped by expert into row tiles
 //   moe_gemm       one projection of every expert over its own rows (gather on the way in, activation or routing weight on
 //                  the way out); moe_fewrows does the same for a handful of pairs with one warp per output
@@ -115,6 +116,7 @@ __device__ __forceinline__ float act_apply(float z, int act) {
     case LIA_ACT_SILU: return z / (1.0f + expf(-z));
     case LIA_ACT_GELU_ERF: return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
     case LIA_ACT_GELU_TANH: return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
+    case LIA_ACT_RELU_SQUARED: return fmaxf(z, 0.f) * fmaxf(z, 0.f);
     default: return z;
   }
 }
@@ -152,11 +154,12 @@ __global__ void gated_act_kernel(const T* __restrict__ in, int ld, int up_off, T
 // One warp per token: softmax over E logits (fp32), or a sigmoid of each (`sigmoid`), then `top` rounds of arg-max (lowest
 // index on ties) over the scores plus an optional per-expert correction that takes part in the choice only; a chosen expert's
 // weight is its plain score, divided by their sum (+ 1e-20) when `renorm` is set.  Sigmoid scores without a correction are
-// compared by their logits (the same order, also where the scores round to 1).
+// compared by their logits (the same order, also where the scores round to 1).  groups > 1: the experts form that many equal runs of
+// neighbours, a run ranks by its largest choice score (lowest index on ties), and only experts of the `keep` best runs can be chosen.
 __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ correction,
                                                           int* __restrict__ idx, float* __restrict__ wt, int M, int E, int top, int renorm,
-                                                          int sigmoid) {
-  extern __shared__ float sc[];          // [4 warps][2][E]: scores, choice scores
+                                                          int sigmoid, int groups, int keep) {
+  extern __shared__ float sc[];          // [4 warps][2][E]: scores, choice scores; then [4 warps][groups]: the groups' best
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row = blockIdx.x * 4 + warp;
   if (row >= M) return;
@@ -185,6 +188,23 @@ __global__ void __launch_bounds__(128) router_topk_kernel(const float* __restric
     }
   }
   __syncwarp();
+  if (groups > 1 && keep < groups) {
+    float* best_of = sc + 8 * E + warp * groups;
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float b = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, ch[e]);
+      best_of[g] = b;
+    }
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {           // a group stays if fewer than `keep` rank ahead of it
+      const int g = e / per;
+      int ahead = 0;
+      for (int o = 0; o < groups; ++o) ahead += best_of[o] > best_of[g] || (best_of[o] == best_of[g] && o < g);
+      if (ahead >= keep) ch[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
   float chosen_sum = 0.f;
   for (int t = 0; t < top; ++t) {
     float best = -INFINITY;
@@ -485,7 +505,7 @@ extern "C" int lia_gated_act_weighted(const void* in, int ld, int up_off, void* 
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(in && out && M > 0 && F > 0 && ld >= F && (up_off < 0 || (up_off >= F && ld >= up_off + F)), "lia_gated_act: bad arguments");
   LIA_CHECK_ARG((perm == nullptr) == (wt == nullptr), "lia_gated_act: a row order and routing weights go together");
-  LIA_CHECK_ARG(act >= LIA_ACT_NONE && act <= LIA_ACT_GELU_TANH, "lia_gated_act: unknown activation %d", act);
+  LIA_CHECK_ARG((act >= LIA_ACT_NONE && act <= LIA_ACT_GELU_TANH) || act == LIA_ACT_RELU_SQUARED, "lia_gated_act: unknown activation %d", act);
   const unsigned blocks = capped_blocks((size_t)M * F);
   if (act_f32) gated_act_kernel<float><<<blocks, 256, 0, stream>>>(reinterpret_cast<const float*>(in), ld, up_off, reinterpret_cast<float*>(out), M, F, act, perm, wt);
   else gated_act_kernel<bf16><<<blocks, 256, 0, stream>>>(reinterpret_cast<const bf16*>(in), ld, up_off, reinterpret_cast<bf16*>(out), M, F, act, perm, wt);
@@ -505,11 +525,19 @@ extern "C" int lia_router_topk_ext(const float* logits, const float* correction,
 // ldl: row stride of the logits (a row may hold more than the experts' logits); sigmoid != 0: scores are sigmoids, not a softmax
 extern "C" int lia_router_topk_scored(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int* idx, float* wt, int M,
                                       int E, int top, lia_stream_t stream_) {
+  return lia_router_topk_grouped(logits, ldl, correction, renorm, sigmoid, 1, 1, idx, wt, M, E, top, stream_);
+}
+
+// groups > 1: only the experts of the `keep` best of that many equal groups of neighbours can be chosen (a group's score is its best expert's)
+extern "C" int lia_router_topk_grouped(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int groups, int keep, int* idx,
+                                       float* wt, int M, int E, int top, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(logits && idx && wt && M > 0 && E > 0 && top > 0 && top <= E && E <= 2048 && ldl >= E, "lia_router_topk: bad arguments (E=%d top=%d)", E, top);
-  const size_t smem = (size_t)8 * E * sizeof(float);
+  LIA_CHECK_ARG(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (E / groups),
+                "lia_router_topk: %d experts, %d of %d groups, %d chosen", E, keep, groups, top);
+  const size_t smem = ((size_t)8 * E + 4 * groups) * sizeof(float);
   if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(router_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  router_topk_kernel<<<(M + 3) / 4, 128, smem, stream>>>(logits, ldl, correction, idx, wt, M, E, top, renorm, sigmoid);
+  router_topk_kernel<<<(M + 3) / 4, 128, smem, stream>>>(logits, ldl, correction, idx, wt, M, E, top, renorm, sigmoid, groups, keep);
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }

@@ -492,7 +492,7 @@ def latent_attn(qa, cache, meta, gate, out, H, kv_rank, rot, scale, max_ctx=0, w
 # Models whose sublayers sit between layer norms on a 32-bit residual stream: decay / delta-rule recurrences, sliding-window
 # attention with grouped key/value heads, dense and mixture-of-experts feed-forwards.  (Not in the reference either.)
 # ------------------------------------------------------------------------------------------------------------------
-ACT_NONE, ACT_RELU, ACT_SILU, ACT_GELU_ERF, ACT_GELU_TANH, ACT_CLAMPED_SWISH = 0, 1, 2, 3, 4, 5
+ACT_NONE, ACT_RELU, ACT_SILU, ACT_GELU_ERF, ACT_GELU_TANH, ACT_CLAMPED_SWISH, ACT_RELU_SQUARED = 0, 1, 2, 3, 4, 5, 6
 I32 = torch.int32
 
 
@@ -558,10 +558,11 @@ def gated_act(inp, F, out, act, up_off=-1, perm=None, wt=None):
     return out
 
 
-def router_topk(logits, top, idx, wt, correction=None, renorm=True, sigmoid=False):
+def router_topk(logits, top, idx, wt, correction=None, renorm=True, sigmoid=False, groups=1, keep=1):
     """Scores of the experts -- a softmax over their logits or (``sigmoid``) the sigmoid of each --, the ``top`` largest and their
     weights: idx int32 [M, top], wt fp32.  ``correction`` [E] is added to the scores for the choice only; ``renorm`` divides the
-    chosen scores by their sum.  ``logits`` may be the left columns of a wider buffer."""
+    chosen scores by their sum.  ``logits`` may be the left columns of a wider buffer.  ``groups`` > 1: the experts form that many equal
+    groups of neighbours and only those of the ``keep`` groups with the best best expert can be chosen."""
     ldl = _rowmajor(logits, "logits")
     _req(idx, "idx", I32); _req(wt, "wt", F32)
     M, E = logits.shape
@@ -571,8 +572,8 @@ def router_topk(logits, top, idx, wt, correction=None, renorm=True, sigmoid=Fals
         raise _lib.LiaError("router_topk: idx and wt must be [M, top], the correction [E]")
     if correction is not None:
         _req(correction, "correction", F32)
-    check(_lib.load().lia_router_topk_scored(_p(logits), ldl, _p(correction), int(renorm), int(sigmoid), _p(idx), _p(wt), M, E, top, _stream()),
-          "lia_router_topk")
+    check(_lib.load().lia_router_topk_grouped(_p(logits), ldl, _p(correction), int(renorm), int(sigmoid), int(groups), int(keep), _p(idx), _p(wt), M, E, top,
+                                              _stream()), "lia_router_topk")
     count_launches()
 
 
@@ -1016,3 +1017,138 @@ def embed_bigram_pos(ids, table, meta, x, bigram=None, hashing=None, tokens=None
                                            float(eps), _stream()), "lia_embed_bigram_pos")
     count_launches()
     return x
+
+
+# ------------------------------------------------------------------------------------------------------------------
+# Designs that keep several residual streams and run two mixers side by side: a state-space dual recurrence, a gated linear
+# recurrent unit.  (Not in the reference either.)
+# ------------------------------------------------------------------------------------------------------------------
+def _stream_shapes(name, x, W, S, vectors):
+    _req(x, "x", F32)
+    if x.dim() != 3 or tuple(x.shape[1:]) != (S, W):
+        raise _lib.LiaError(f"{name}: x must be [rows, {S}, {W}]")
+    for t, n, size in vectors:
+        if t is not None and _req(t, n, F32).numel() != size:
+            raise _lib.LiaError(f"{name}: {n} must be fp32 of {size} numbers")
+
+
+def streams_update(x, y, mix, w_out, w_in, w, h, eps, branch_norms=None, y2=None, scale=1.0):
+    """The update of a residual kept as S streams ``x`` [rows, S, W] (fp32, in place) by a sublayer's output, and what the next
+    sublayer reads:  v = y, or with ``branch_norms`` = (w_y, w_y2) scale * (N(y; w_y) + N(y2; w_y2));
+    x[t] = sum_s mix[s, t] x[s] + w_out[t] v from the old streams (``y`` None: unchanged);  h = N(sum_s w_in[s] x[s]; w) (``h`` None: not
+    made), N(z; w) = w z / rms(z)."""
+    rows, S, W = x.shape
+    w_y, w_y2 = branch_norms if branch_norms is not None else (None, None)
+    _stream_shapes("streams_update", x, W, S, ((mix if y is not None else None, "mix", S * S), (w_out if y is not None else None, "w_out", S),
+                                               (w_in if h is not None else None, "w_in", S), (w if h is not None else None, "w", W),
+                                               (w_y, "w_y", W), (w_y2 if y2 is not None else None, "w_y2", W)))
+    for t, n in ((y, "y"), (y2, "y2"), (h, "h")):
+        if t is not None and not (t.is_cuda and t.is_contiguous() and tuple(t.shape) == (rows, W)):
+            raise _lib.LiaError(f"streams_update: {n} must be a contiguous CUDA [{rows}, {W}] tensor")
+    if y2 is not None and y2.dtype != y.dtype:
+        raise _lib.LiaError("streams_update: both branches must have one type")
+    check(_lib.load().lia_streams_update(_p(x), _p(y), _f32(y) if y is not None else 0, _p(w_y), _p(y2), _p(w_y2) if y2 is not None else None, float(scale), _p(mix), _p(w_out),
+                                         _p(w_in), _p(w), _p(h), _f32(h) if h is not None else 0, rows, S, W, float(eps), _stream()), "lia_streams_update")
+    count_launches()
+    return x
+
+
+def streams_embed(ids, table, x, w_in, w, h, eps):
+    """All S streams of row r = table[ids[r]] (fp32); h = N(sum_s w_in[s] x[s]; w), ``h`` (may be None) of the table's dtype."""
+    _req(ids, "ids", torch.int64); _dev(table, "table")
+    rows, S, W = x.shape
+    _stream_shapes("streams_embed", x, W, S, ((w_in if h is not None else None, "w_in", S), (w if h is not None else None, "w", W)))
+    if h is not None and not (h.is_contiguous() and tuple(h.shape) == (rows, W) and h.dtype == table.dtype):
+        raise _lib.LiaError("streams_embed: h must be a contiguous [rows, W] tensor of the table's dtype")
+    check(_lib.load().lia_streams_embed(_p(ids), _p(table), _f32(table), _p(x), _p(w_in), _p(w), _p(h), rows, S, W, table.shape[0], float(eps), _stream()),
+          "lia_streams_embed")
+    count_launches()
+    return x
+
+
+def streams_gather(x, rows, w, h, eps):
+    """h[r] = N(sum_s x[rows[r], s]; w): the final norm of the rows whose logits are wanted."""
+    _req(rows, "rows", I32)
+    n, W = h.shape
+    _stream_shapes("streams_gather", x, W, x.shape[1], ((w, "w", W),))
+    if rows.numel() != n or not h.is_contiguous():
+        raise _lib.LiaError("streams_gather: a row index per row of h")
+    check(_lib.load().lia_streams_gather(_p(x), _p(rows), _p(w), _p(h), _f32(h), n, x.shape[1], W, float(eps), _stream()), "lia_streams_gather")
+    count_launches()
+    return h
+
+
+def silu_gate_norm(o, z, w, out, groups, eps):
+    """out = w * g / rms(g) with g = o * silu(z), the root mean square taken over each of ``groups`` equal parts of a row."""
+    _req(o, "o", F32)
+    ldz = _rowmajor(z, "z")
+    M, F = o.shape
+    if tuple(z.shape) != (M, F) or not (out.is_cuda and out.is_contiguous() and tuple(out.shape) == (M, F) and out.dtype == z.dtype) or _req(w, "w", F32).numel() != F:
+        raise _lib.LiaError("silu_gate_norm: z an [M, F] slice, out a contiguous [M, F] tensor of its dtype, w fp32 [F]")
+    check(_lib.load().lia_silu_gate_norm(_p(o), _p(z), ldz, _p(w), _p(out), _f32(out), M, F, int(groups), float(eps), _stream()), "lia_silu_gate_norm")
+    count_launches()
+    return out
+
+
+def conv_act(y, col0, wconv, out, batch, state=None, in_bias=None, bias=None, act=ACT_NONE, dt_col=0, dt_bias=None, a_log=None, gates=None):
+    """A short causal convolution along the sequence on the columns [col0, col0 + C) of a projection's output ``y``: out [M, C] (a left
+    part of a wider fp32 buffer is fine) = act(sum over the taps of wconv [C, taps] + bias), inputs y + in_bias, zero before the
+    sequence's start.  ``state`` [slots, taps - 1, C] holds the inputs before each portion and is moved on.  With ``gates`` [M, 2H] the
+    columns [dt_col, dt_col + H) become gates = dt | g: dt = softplus(y + dt_bias), g = exp(-exp(a_log) dt)."""
+    ld, ldo = _rowmajor(y, "y"), _rowmajor(out, "out")
+    C, taps = _req(wconv, "wconv", F32).shape
+    M = y.shape[0]
+    for t, n, size in ((in_bias, "in_bias", C), (bias, "bias", C)):
+        if t is not None and _req(t, n, F32).numel() != size:
+            raise _lib.LiaError(f"conv_act: {n} must be fp32 [{size}]")
+    if taps > 1 and (state is None or tuple(_req(state, "state", F32).shape[1:]) != (taps - 1, C)):
+        raise _lib.LiaError("conv_act: the state must be fp32 [slots, taps - 1, C]")
+    if out.dtype != F32 or tuple(out.shape) != (M, C):
+        raise _lib.LiaError(f"conv_act: out must be fp32 [{M}, {C}]")
+    H = 0
+    if gates is not None:
+        H = _req(gates, "gates", F32).shape[1] // 2
+        if tuple(gates.shape) != (M, 2 * H) or _req(dt_bias, "dt_bias", F32).numel() != H or _req(a_log, "a_log", F32).numel() != H:
+            raise _lib.LiaError("conv_act: gates [M, 2H], dt_bias and a_log [H]")
+    n = batch.segs.shape[0]
+    check(_lib.load().lia_conv_act(_p(y), _f32(y), ld, int(col0), C, _p(in_bias), _p(wconv), _p(bias), taps, act, _p(state) if taps > 1 else None,
+                                   _p(batch.meta), _p(batch.segs), n, _p(out), ldo, M, int(dt_col), H, _p(dt_bias) if H else None,
+                                   _p(a_log) if H else None, _p(gates), _stream()), "lia_conv_act")
+    count_launches(2 if taps > 1 and n != M else 1)
+    return out
+
+
+def ssd_scan(xbc, gates, D, state_S, segs, H, G, N, vdim, o):
+    """State-space dual recurrence S = g S + dt B x^T, o = S^T C + D x over every portion of the step (csrc/linear_scan.cu).  ``xbc`` fp32
+    [M, H vdim + 2 G N] = x | B | C; gates [M, 2H] = dt | g; state_S [slots, H, vdim, N]."""
+    ld = _rowmajor(xbc, "xbc")
+    M, inner = xbc.shape[0], H * vdim
+    for t, n in ((gates, "gates"), (D, "D"), (state_S, "state_S"), (o, "o")):
+        _req(t, n, F32)
+    _req(segs, "segs", I32)
+    if xbc.dtype != F32 or xbc.shape[1] != inner + 2 * G * N or tuple(gates.shape) != (M, 2 * H) or D.numel() != H or tuple(o.shape) != (M, inner) \
+            or tuple(state_S.shape[1:]) != (H, vdim, N):
+        raise _lib.LiaError("ssd_scan: shapes do not agree")
+    check(_lib.load().lia_ssd_scan(_p(xbc[:, inner:]), _p(xbc[:, inner + G * N:]), _p(xbc), ld, _p(gates), _p(D), _p(state_S), _p(segs), segs.shape[0], H, G, N,
+                                   vdim, _p(o), _stream()), "lia_ssd_scan")
+    count_launches()
+    return o
+
+
+def rglru_scan(u, z, z_bias, c, y, y_bias, state, segs, blocks, out):
+    """Gated linear recurrent unit over every portion of the step (csrc/linear_scan.cu): log a = c sigmoid(r + bias),
+    S = a S + sqrt(1 - a^2) sigmoid(i + bias) u, out = S * gelu_tanh(y + y_bias).  u fp32 [M, width]; z fp32 [M, 2 width] = r | i block by
+    block; state [slots, width]; ``y`` a column slice and ``out`` [M, width] of one dtype."""
+    for t, n in ((u, "u"), (z, "z"), (z_bias, "z_bias"), (c, "c"), (state, "state"), (y_bias, "y_bias")):
+        if t is not None:
+            _req(t, n, F32)
+    _req(segs, "segs", I32)
+    ldy = _rowmajor(y, "y")
+    M, width = u.shape
+    if tuple(z.shape) != (M, 2 * width) or z_bias.numel() != 2 * width or c.numel() != width or tuple(y.shape) != (M, width) or tuple(state.shape[1:]) != (width,) \
+            or width % blocks or not (out.is_cuda and out.is_contiguous() and tuple(out.shape) == (M, width) and out.dtype == y.dtype):
+        raise _lib.LiaError("rglru_scan: shapes do not agree")
+    check(_lib.load().lia_rglru_scan(_p(u), _p(z), _p(z_bias), _p(c), _p(y), _f32(y), ldy, _p(y_bias), _p(state), _p(segs), segs.shape[0], width, int(blocks),
+                                     _p(out), _stream()), "lia_rglru_scan")
+    count_launches()
+    return out
