@@ -42,6 +42,11 @@ def _pazivik():
     return PazivikForCausalLM
 
 
+def _sekenex():
+    from .modeling_sekenex import SekenexForCausalLM
+    return SekenexForCausalLM
+
+
 register("OPTForCausalLM", _opt)
 register("opt", _opt)
 register("Davasun", _davasun)
@@ -54,6 +59,8 @@ register("Zatusun", _zatusun)
 register("ZatusunForCausalLM", _zatusun)
 register("Pazivik", _pazivik)
 register("PazivikForCausalLM", _pazivik)
+register("Sekenex", _sekenex)
+register("SekenexForCausalLM", _sekenex)
 
 
 def architecture_of(path):

@@ -5,8 +5,9 @@ the cache a layer's own or an earlier layer's), linear attention with a fixed
 decay per head, linear attention with a forget gate per channel, the gated delta rule behind a short convolution, differential
 attention (two softmax maps over shared values, subtracted) under a chunked or sliding mask, sliding-window attention with grouped key/value heads, attention over the whole history with a sink in the
 softmax (behind an optional bias, convolution, norm, temperature and rotation of its inputs, with a distance bias, a blend of
-values across layers and an output gate), and the feed-forwards -- clamped gated, plain gated with any activation, one with a
-polynomial activation between norms, and a routed mixture of experts (plain or gated experts weighed on the way out or on the way in, a
+values across layers and an output gate), state-space duality (Mamba-2), a gated linear recurrent unit (Griffin's recurrent block), two mixers
+side by side, and the feed-forwards -- clamped gated, plain gated with any activation, one with a
+polynomial activation between norms, and a routed mixture of experts (chosen among all experts or among the best groups of them; plain or gated experts weighed on the way out or on the way in, a
 shared expert with or without a gate, experts that hand the token back).  Each object owns its (fused) weights,
 registers its per-sequence state with a ``seq_state.SlotState`` and runs one step over a batch of portions
 (``StepBatch``) through the kernels of ``ops``.
@@ -40,11 +41,12 @@ class StepBatch:
 
 class Linear:
     """y = x @ W.T for one or several weight matrices stacked by rows (one launch, outputs side by side; each block's
-    first column is a multiple of 8 so that every slice stays 16-byte aligned in bf16)."""
+    first column is a multiple of 8 so that every slice stays 16-byte aligned in bf16).  ``pad``: so does the whole output's width, for outputs
+    that are read slice by slice (the last columns are zeros)."""
 
     _gemm_ws = {}
 
-    def __init__(self, weights, dtype, device):
+    def __init__(self, weights, dtype, device, pad=False):
         ws = [w.to(device=device, dtype=dtype) for w in weights]
         self.K = ws[0].shape[1]
         self.offsets, n = [], 0
@@ -52,7 +54,7 @@ class Linear:
             self.offsets.append(_pad8(n))
             n = self.offsets[-1] + w.shape[0]
         self.sizes = [w.shape[0] for w in ws]
-        self.N = n
+        self.N = n = _pad8(n) if pad else n
         self.weight = torch.zeros(n, self.K, dtype=dtype, device=device)
         for o, w in zip(self.offsets, ws):
             self.weight[o:o + w.shape[0]] = w
@@ -505,16 +507,17 @@ def scaled_rotary_freq(dims, base, scaling=None):
 
 
 class SinkAttentionMixer:
-    """Causal softmax attention over the whole history with grouped key/value heads and one learned sink per head in the
-    softmax's denominator (a term without key or value).  Everything else is an option, so that designs which differ in them
-    share the mixer:
+    """Causal softmax attention over the whole history with grouped key/value heads.  Everything else is an option, so that designs which
+    differ in them share the mixer:
+      ``sink``     True: one learned sink per head joins the softmax's denominator (a term without key or value);
       ``biases``   q, k, v projections with biases ("q.b", ...);
       ``taps``     a short causal convolution along the sequence on every channel of q, k, v right after the projection ("q.conv"
                    [channels, taps], ...; None: no convolution); the last taps - 1 projected rows are per-sequence state;
       ``norm``     "whole": one RMS norm over all of q and one over all of k ("q.norm" [H*dim], "k.norm" [G*dim]);
                    "head": per head with a weight [dim] shared by the heads;
       ``q_temp``   (coef, every): q times 1 + coef * ln(floor((pos + 1) / every) + 1);
-      ``rot``      {"dims", "base", "scaling"}: the first ``dims`` channels of every q and k head turn in pairs (2i, 2i+1);
+      ``rot``      {"dims", "base", "scaling"}: the first ``dims`` channels of every q and k head turn in pairs (2i, 2i+1), or
+                   (``rot_halves``) in pairs (i, i + dims/2);
       ``slopes``   [H]: every position between query and key costs head h slopes[h] of the score;
       ``v_mix``    "publish": this layer's values are left in the step's scratch for later layers; "blend": v becomes
                    (1 - vmix) v + vmix v_published before it is cached;
@@ -525,7 +528,7 @@ class SinkAttentionMixer:
     model's dtype (csrc/window_attn.cu)."""
 
     def __init__(self, w, heads, kv_heads, dim, vdim, scale, norm_eps, dtype, device, norm=None, biases=False, taps=None, q_temp=None, rot=None,
-                 slopes=None, v_mix=None, gate=None, ride_along=()):
+                 slopes=None, v_mix=None, gate=None, ride_along=(), sink=True, rot_halves=False):
         if heads % kv_heads:
             raise ValueError(f"{heads} heads do not divide into {kv_heads} key/value heads")
         if norm not in (None, "whole", "head") or gate not in (None, "head", "channel") or v_mix not in (None, "publish", "blend"):
@@ -536,7 +539,7 @@ class SinkAttentionMixer:
         self.channels = nq + nk + nv
         stacked = [w["q"], w["k"], w["v"]] + ([w["g"]] if gate == "channel" else []) + list(ride_along)
         self.n_ride, self.gate = len(ride_along), gate
-        self.proj = Linear(stacked, dtype, device)
+        self.proj = Linear(stacked, dtype, device, pad=True)
         f32 = dict(device=device, dtype=F32)
         self.bias = torch.cat([w["q.b"], w["k.b"], w["v.b"]]).to(**f32).contiguous() if biases else None
         self.w_conv = torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]], 0).to(**f32).contiguous() if taps else None
@@ -544,7 +547,7 @@ class SinkAttentionMixer:
         self.q_norm = w["q.norm"].to(**f32).contiguous() if norm else None
         self.k_norm = w["k.norm"].to(**f32).contiguous() if norm else None
         self.temp_coef, self.temp_every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
-        self.rot_dims, self.freq, self.rot_mag = 0, None, 1.0
+        self.rot_dims, self.freq, self.rot_mag, self.rot_halves = 0, None, 1.0, bool(rot_halves)
         if rot:
             self.rot_dims = int(rot["dims"])
             if self.rot_dims % 2 or not 0 < self.rot_dims <= dim:
@@ -552,7 +555,7 @@ class SinkAttentionMixer:
             f, self.rot_mag = scaled_rotary_freq(self.rot_dims, rot["base"], rot.get("scaling"))
             self.freq = f.to(device).contiguous()
         self.slopes = torch.tensor([float(x) for x in slopes], dtype=torch.float64).to(**f32) if slopes is not None else None
-        self.sink = w["sink"].to(**f32).contiguous()
+        self.sink = w["sink"].to(**f32).contiguous() if sink else None
         self.vmix_mode = {None: ops.VMIX_NONE, "publish": ops.VMIX_PUBLISH, "blend": ops.VMIX_BLEND}[v_mix]
         self.vmix = float(w["vmix"]) if v_mix == "blend" else 0.0
         self.w_gate = w["g"].to(device=device, dtype=dtype).contiguous() if gate == "head" else None
@@ -589,7 +592,7 @@ class SinkAttentionMixer:
         offs = self.proj.offsets[:3]
         ops.qkv_prep(y, offs, batch.meta, q, kc, vc, H, G, self.dim, self.vdim, self.eps, bias=self.bias, wconv=self.w_conv, conv_state=conv,
                      taps=self.taps, norm_mode=self.norm_mode, qnorm_w=self.q_norm, knorm_w=self.k_norm, temp_coef=self.temp_coef,
-                     temp_every=self.temp_every, freq=self.freq, rot_dims=self.rot_dims, rot_mag=self.rot_mag, vmix_mode=self.vmix_mode,
+                     temp_every=self.temp_every, freq=self.freq, rot_dims=self.rot_dims, rot_halves=self.rot_halves, rot_mag=self.rot_mag, vmix_mode=self.vmix_mode,
                      vmix=self.vmix, v_first=v_first)
         if self.taps > 1:
             ops.conv_state_update(y, offs, H * self.dim, G * self.vdim, conv, batch.segs, self.taps, nk=G * self.dim)
@@ -597,6 +600,108 @@ class SinkAttentionMixer:
         ops.window_attn(q, kc, vc, batch.meta, None, o, H, G, self.dim, self.vdim, 0, self.scale, 0.0, nseg=batch.segs.shape[0],
                         max_ctx=batch.max_ctx, slopes=self.slopes, sink=self.sink, gate=gate, gate_per_head=self.gate == "head")
         return self.out(o)
+
+
+class GatedRecurrentMixer:
+    """Griffin's recurrent block: y = gelu_tanh(Wy h + by) beside u = conv(Wx h + bx), a short causal convolution with a bias per channel; in each of
+    ``blocks`` equal parts of u two gates r = sigmoid(Ra u + ra), i = sigmoid(Ri u + ri); log a = -decay * r * softplus(lam),
+    S = a S + sqrt(1 - a^2) i u (csrc/linear_scan.cu), output Wo (S * y).  u, the gates, the decay and the state are fp32.
+    ``projected``: the caller's stacked projection carries Wy and Wx (the weights ``ride_along``) and hands their outputs in."""
+
+    def __init__(self, w, width, blocks, taps, dtype, device, decay=8.0, projected=False):
+        if width % blocks:
+            raise ValueError(f"{width} channels do not divide into {blocks} blocks")
+        self.width, self.blocks, self.taps, self.dtype = width, blocks, int(taps), dtype
+        n = width // blocks
+        f32 = dict(device=device, dtype=F32)
+        self.proj = None if projected else Linear([w["y"], w["x"]], dtype, device, pad=True)
+        self.y_bias, self.x_bias = w["y.b"].to(**f32).contiguous(), w["x.b"].to(**f32).contiguous()
+        self.w_conv, self.conv_bias = w["conv"].to(**f32).contiguous(), w["conv.b"].to(**f32).contiguous()
+        self.w_gates = torch.cat([w["ra"], w["ri"]], 1).to(device=device, dtype=dtype).contiguous()            # [blocks, r | i, n]
+        self.gate_bias = torch.cat([w["ra.b"], w["ri.b"]], 1).to(**f32).contiguous()
+        lam = w["lam"].to(torch.float64)
+        self.c = (-float(decay) * torch.nn.functional.softplus(lam, threshold=100.0)).to(**f32).contiguous()
+        self.out = Linear([w["o"]], dtype, device)
+        self.n = n
+
+    @staticmethod
+    def ride_along(w):
+        return [w["y"], w["x"]]
+
+    def new_state(self, slots):
+        return (slots.add_recurrent((self.width,)), slots.add_recurrent((max(self.taps - 1, 1), self.width)))
+
+    def __call__(self, h, batch, state, projected=None):
+        S, conv = state
+        M, W, n = h.shape[0], self.width, self.n
+        if projected is None:
+            p = self.proj(h)
+            projected = [self.proj.part(p, 0), self.proj.part(p, 1)]
+        y, x = projected
+        u = torch.empty(M, W, dtype=F32, device=h.device)
+        ops.conv_act(x, 0, self.w_conv, u, batch, state=conv, in_bias=self.x_bias, bias=self.conv_bias)
+        z = torch.empty(M, 2 * W, dtype=F32, device=h.device)
+        ops.linear_plain(u, self.w_gates, z, batch=self.blocks, a_batch_stride=n, w_batch_stride=2 * n * n, out_batch_stride=2 * n, n=2 * n, k=n)
+        o = torch.empty(M, W, dtype=self.dtype, device=h.device)
+        ops.rglru_scan(u, z, self.gate_bias, self.c, y, self.y_bias, S, batch.segs, self.blocks, o)
+        return self.out(o)
+
+
+class ParallelMixer:
+    """Two mixers on one input, side by side: half the sum of their outputs, each first RMS-normed with a plain weight.  ``left`` is built with
+    the projections of ``right`` riding along on its own (one GEMM for both) if ``shared_projection``.  The call returns the two
+    outputs; ``branch_norms`` and ``branch_scale`` say how the residual update that follows joins them (``ops.streams_update``)."""
+
+    branch_scale = 0.5
+
+    def __init__(self, left, right, left_norm, right_norm, device, shared_projection=True):
+        self.left, self.right, self.shared_projection = left, right, shared_projection
+        self.branch_norms = tuple(t.to(device=device, dtype=F32).contiguous() for t in (left_norm, right_norm))
+
+    def new_state(self, slots):
+        return self.left.new_state(slots), self.right.new_state(slots)
+
+    def __call__(self, h, batch, state):
+        extras = [] if self.shared_projection else None
+        left = self.left(h, batch, state[0], extras) if self.shared_projection else self.left(h, batch, state[0])
+        return left, (self.right(h, batch, state[1], extras) if self.shared_projection else self.right(h, batch, state[1]))
+
+
+class StateSpaceMixer:
+    """Mamba-2's mixer (state-space duality): Win h = z | x | B | C | dt; x, B and C pass a short causal convolution with a bias per channel and
+    SiLU; dt = softplus(dt + dt_bias); per head S = exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x (csrc/linear_scan.cu; the heads share
+    B and C in ``groups``); y * silu(z) RMS-normed in ``norm_groups`` equal parts with a plain weight, then Wo.  Step sizes, decays, state and
+    sums are fp32."""
+
+    def __init__(self, w, heads, vdim, state, groups, norm_groups, taps, norm_eps, dtype, device):
+        inner = heads * vdim
+        if heads % groups or inner % norm_groups:
+            raise ValueError(f"{heads} heads of {vdim} in {groups} groups, {norm_groups} parts of the norm")
+        self.H, self.vdim, self.N, self.G, self.norm_groups = heads, vdim, state, groups, norm_groups
+        self.inner, self.C, self.taps, self.eps, self.dtype = inner, inner + 2 * groups * state, int(taps), float(norm_eps), dtype
+        w_in = w["in"]
+        self.proj = Linear([w_in[:inner], w_in[inner:inner + self.C], w_in[inner + self.C:]], dtype, device, pad=True)
+        f32 = dict(device=device, dtype=F32)
+        self.w_conv, self.conv_bias = w["conv"].to(**f32).contiguous(), w["conv.b"].to(**f32).contiguous()
+        self.dt_bias, self.a_log, self.D, self.norm_w = (w[k].to(**f32).contiguous() for k in ("dt_bias", "A_log", "D", "norm"))
+        self.out = Linear([w["o"]], dtype, device)
+
+    def new_state(self, slots):
+        return (slots.add_recurrent((self.H, self.vdim, self.N)), slots.add_recurrent((max(self.taps - 1, 1), self.C)))
+
+    def __call__(self, h, batch, state):
+        S, conv = state
+        M, dev = h.shape[0], h.device
+        y = self.proj(h)
+        xbc = torch.empty(M, (self.C + 3) // 4 * 4, dtype=F32, device=dev)[:, :self.C]         # rows stay 16-byte aligned
+        gates = torch.empty(M, 2 * self.H, dtype=F32, device=dev)
+        ops.conv_act(y, self.proj.offsets[1], self.w_conv, xbc, batch, state=conv, bias=self.conv_bias, act=ops.ACT_SILU, dt_col=self.proj.offsets[2],
+                     dt_bias=self.dt_bias, a_log=self.a_log, gates=gates)
+        o = torch.empty(M, self.inner, dtype=F32, device=dev)
+        ops.ssd_scan(xbc, gates, self.D, S, batch.segs, self.H, self.G, self.N, self.vdim, o)
+        on = torch.empty(M, self.inner, dtype=self.dtype, device=dev)
+        ops.silu_gate_norm(o, self.proj.part(y, 0), self.norm_w, on, self.norm_groups, self.eps)
+        return self.out(on)
 
 
 class PolyNormMLP:
@@ -658,7 +763,8 @@ class MoEFeedForward:
     with ``renorm`` the weights equal a softmax restricted to the selected experts' logits; ``score`` = "sigmoid": an expert's score is
     the sigmoid of its logit; ``weigh`` = "input": the weight multiplies what goes into the expert (expert(w * h)) instead of what
     comes out; a shared expert (optional) runs for every token and is added, times sigmoid(``shared_gate`` h) if that weight [1, W] is
-    given (its logit rides on the router's projection).  ``experts_w``: list of {"up", "down"[, "gate"]} per expert.  The (token, choice) pairs are
+    given (its logit rides on the router's projection).  ``groups`` = (count, keep): the experts form ``count`` equal groups of neighbours, and only
+    experts of the ``keep`` groups with the best best score can be chosen.  ``experts_w``: list of {"up", "down"[, "gate"]} per expert.  The (token, choice) pairs are
     grouped by expert on the device (no host round trip) and each projection runs as one grouped launch; a handful of pairs
     (decoding) take the form with one warp per output instead.  The result is fp32."""
 
@@ -666,7 +772,7 @@ class MoEFeedForward:
     TENSOR_CORE_PAIRS = 512   # from here (bf16, sizes that are multiples of 8): every expert's rows through the tensor-core GEMM
 
     def __init__(self, router_w, experts_w, top, ff, act, shared, dtype, device, correction=None, renorm=True, identity=0, act_params=(0.0, 0.0),
-                 score="softmax", weigh="output", shared_gate=None):
+                 score="softmax", weigh="output", shared_gate=None, groups=None):
         if score not in ("softmax", "sigmoid") or weigh not in ("output", "input"):
             raise ValueError(f"unknown option: score={score!r} weigh={weigh!r}")
         if shared_gate is not None and shared is None:
@@ -680,6 +786,9 @@ class MoEFeedForward:
         self.R = self.E + self.identity                          # router outputs
         if not 1 <= self.top <= self.R or self.E < 1 or router_w.shape[0] != self.R:
             raise ValueError(f"top = {top} of {self.E} experts + {self.identity} identity experts, router of {router_w.shape[0]} outputs")
+        self.groups, self.keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
+        if self.R % self.groups or not 1 <= self.keep <= self.groups or self.top > self.keep * (self.R // self.groups):
+            raise ValueError(f"cannot choose {self.top} of {self.R} experts in the {self.keep} best of {self.groups} groups")
         if shared_gate is not None:
             router_w = torch.cat([router_w, shared_gate], 0)     # one launch: the experts' logits, then the shared expert's
         self.router = router_w.to(device=device, dtype=dtype).contiguous()
@@ -741,7 +850,8 @@ class MoEFeedForward:
         ops.linear_small(h if router_input is None else router_input, self.router, None, logits, ops.GATE_NONE)
         idx = torch.empty(M, top, dtype=torch.int32, device=dev)
         wt = torch.empty(M, top, dtype=F32, device=dev)
-        ops.router_topk(logits[:, :R], top, idx, wt, correction=self.correction, renorm=self.renorm, sigmoid=self.sigmoid)
+        ops.router_topk(logits[:, :R], top, idx, wt, correction=self.correction, renorm=self.renorm, sigmoid=self.sigmoid, groups=self.groups,
+                        keep=self.keep)
         shared_gate = logits[:, R:] if self.shared_gated else None
         identity = (idx, self.E, h, wt) if self.identity else None
         pairs = M * top
