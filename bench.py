@@ -70,6 +70,8 @@ def parse():
                     help="instead of the headline workload: the same comparison for Zatusun beside Bebulorn, its closest existing model")
     ap.add_argument("--compare-pazivik", action="store_true",
                     help="instead of the headline workload: the same comparison for Pazivik beside Zatusun, its closest existing model")
+    ap.add_argument("--compare-sekenex", action="store_true",
+                    help="instead of the headline workload: the same comparison for Sekenex beside Bebulorn, its closest existing model")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-parity", action="store_true")
     ap.add_argument("--no-graphs", action="store_true")
@@ -426,6 +428,11 @@ def _main(args, json_out):
         from lia_b200 import bench_compare
         if rank == 0:
             json_out.write(json.dumps(bench_compare.run_pazivik(peaks())) + "\n")
+        return 0
+    if args.compare_sekenex:
+        from lia_b200 import bench_compare
+        if rank == 0:
+            json_out.write(json.dumps(bench_compare.run_sekenex(peaks())) + "\n")
         return 0
     from lia_b200.modeling_opt import get_config
     cfg = get_config(args.model)

@@ -8,6 +8,8 @@ key/value heads on the same attention kernel, dense and mixture-of-experts feed-
 softmax attention and routed experts on the same kernels, a looped block, step-served).
 `bench.py --compare-pazivik`: the same for Pazivik beside Zatusun, the closest existing model (latent attention on the same kernel,
 gated routed experts, pre-norm fp32 stream, step-served).
+`bench.py --compare-sekenex`: the same for Sekenex beside Bebulorn, the closest existing model (matrix-state recurrences behind short
+convolutions, softmax attention with grouped heads on the same kernel, dense feed-forwards and routed experts, step-served).
 
 Each operation of ``ops`` is wrapped for the duration of an instrumented pass: CUDA events around the call, and the
 operation's algorithmic FLOPs and bytes from its arguments.  roofline time = max(FLOPs / peak, bytes / HBM bandwidth)
@@ -87,6 +89,29 @@ def _cost(name, a, kw):
     if name == "poly_norm":
         inp, F, out = a[0], a[1], a[3]
         return 0.0, 2.0 * inp.shape[0] * F * inp.element_size() + _nbytes(out), "mem"
+    if name == "streams_update":
+        x, y, h, y2 = a[0], a[1], a[6], kw.get("y2")
+        return 0.0, 2.0 * _nbytes(x) + _nbytes(y, y2, h), "mem"
+    if name == "streams_embed":
+        table, x, h = a[1], a[2], a[5]
+        return 0.0, _nbytes(x, h) + x.shape[0] * x.shape[2] * table.element_size(), "mem"
+    if name == "streams_gather":
+        x, h = a[0], a[3]
+        return 0.0, h.shape[0] * x.shape[1] * x.shape[2] * 4.0 + _nbytes(h), "mem"
+    if name == "conv_act":
+        y, out, gates = a[0], a[3], kw.get("gates")
+        M, C = out.shape
+        return 0.0, M * C * (y.element_size() + 4.0) + (gates.numel() * (4.0 + y.element_size() / 2) if gates is not None else 0), "mem"
+    if name == "ssd_scan":
+        xbc, gates, S, segs, o = a[0], a[1], a[3], a[4], a[9]
+        H, N, vdim = a[5], a[7], a[8]
+        return 4.0 * xbc.shape[0] * H * N * vdim, 2.0 * segs.shape[0] * H * N * vdim * 4 + xbc.shape[0] * xbc.shape[1] * 4.0 + _nbytes(gates, o), "f32"
+    if name == "rglru_scan":
+        u, z, y, out = a[0], a[1], a[4], a[9]
+        return 0.0, _nbytes(u, z, out) + u.numel() * y.element_size() + 2.0 * a[7].shape[0] * u.shape[1] * 4, "mem"
+    if name == "silu_gate_norm":
+        o, z, out = a[0], a[1], a[3]
+        return 0.0, _nbytes(o, out) + o.numel() * z.element_size(), "mem"
     if name == "moe_gemm":
         x, w, out, idx = a[0], a[1], a[2], a[3]
         pairs, N, K = idx.numel(), w.shape[1], w.shape[2]
@@ -115,7 +140,7 @@ class Instrument:
              "linear_scan", "conv_prep", "conv_state_update", "kv_store", "window_attn", "ln_add_norm", "embed_rows", "ln_gather", "gated_act",
              "router_topk", "moe_plan", "moe_gemm", "moe_gather", "moe_expert_gemms", "moe_combine", "qkv_prep", "gated_rms_add", "poly_norm",
              "embed_scale_pos", "residual_norm", "rms_norm_rows", "sigmoid_mul", "softcap", "forget_gate_prep", "forget_scan", "diff_combine",
-             "latent_store", "embed_bigram_pos")
+             "latent_store", "embed_bigram_pos", "streams_update", "streams_embed", "streams_gather", "conv_act", "ssd_scan", "rglru_scan", "silu_gate_norm")
 
     def __init__(self):
         self.records, self.saved, self.extra = [], {}, {}
@@ -242,10 +267,28 @@ def pazivik_config(width, n_layers):
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}}
 
 
+def sekenex_config(width, n_layers):
+    """Layer sizes of a ~1-3 B model on four residual streams: state-space mixers twice as wide as the model with heads of 64 and a state of 128
+    behind a 4-tap convolution; every fourth layer attention with heads of 128 x 128 on 8 key/value heads (half of each rotated, 3-tap
+    convolutions) beside a recurrent block of the model's width in blocks of 256; feed-forwards alternate between a dense 2.75 x one and 16 experts of
+    0.6875 x (2 chosen, from the 2 best of 4 groups) plus a shared expert of the same size.  Order: state space, parallel, state
+    space, state space."""
+    H = width // 128
+    dense = {"kind": "dense", "ff": width * 11 // 4}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": width * 11 // 16}, "shared": {"ff": width * 11 // 16}}
+    ss = lambda mlp: {"type": "mamba2", "mlp": mlp,  # noqa: E731
+                      "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}}
+    par = {"type": "parallel", "mlp": moe,
+           "mixer": {"left": {"heads": H, "kv_heads": min(8, H), "dim": 128, "vdim": 128, "conv": 3, "rot": {"dims": 64, "base": 500000.0}, "scale": 128 ** -0.5},
+                     "right": {"width": width, "blocks": width // 256, "conv": 4}}}
+    pattern = [ss(dense), par, ss(dense), ss(moe)]
+    return {"architecture": "Sekenex", "vocab": 32000, "width": width, "streams": 4, "layers": [pattern[i % 4] for i in range(n_layers)], "norm": {"eps": 1e-6}}
+
+
 def _window_keys(layers, n_new, ctx_before):
     """Sum over the new rows of the keys inside the first attention layer's window (the whole history where a layer names
     none), and the cached rows those windows span."""
-    first = next((l for l in layers if l["type"].startswith("attention") or (l["type"] == "latent_attention" and "mask" in l["mixer"])), None)
+    first = next((l for l in layers if l["type"].startswith("attention") or l["type"] == "parallel" or (l["type"] == "latent_attention" and "mask" in l["mixer"])), None)
     win = first["mixer"].get("mask", {}).get("size", 1 << 30) if first else 0
     if not win:
         return 0, 0
@@ -334,6 +377,27 @@ def run_zatusun(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=204
     return out
 
 
+def run_sekenex(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=2048, decode_batches=(1, 16), new=16):
+    """Sekenex beside Bebulorn at equal width and depth."""
+    from .modeling_bebulorn import BebulornConfig, BebulornForCausalLM
+    from .modeling_sekenex import SekenexConfig, SekenexForCausalLM
+    dev = torch.device("cuda", 0)
+    props = torch.cuda.get_device_properties(dev)
+    pk = dict(pk, fp32_nominal_tflops=props.multi_processor_count * 128 * 2 * 1.965e9 / 1e12)
+    out = {"peaks": pk, "sizes": []}
+    g = torch.Generator().manual_seed(0)
+    for width in widths:
+        rec = {"width": width, "layers": n_layers, "prompt": prompt, "decode_context": decode_ctx}
+        for name, make in (("sekenex", lambda: SekenexForCausalLM(SekenexConfig.from_dict(sekenex_config(width, n_layers)), dev, BF16)),
+                           ("bebulorn", lambda: BebulornForCausalLM(BebulornConfig.from_dict(bebulorn_config(width, n_layers)), dev, BF16))):
+            m = make().init_weights(seed=1)
+            rec[name] = step_model(m, m.config, pk, g, prompt, decode_ctx, decode_batches, new)
+            del m
+            torch.cuda.empty_cache()
+        out["sizes"].append(rec)
+    return out
+
+
 def run_pazivik(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=2048, decode_batches=(1, 16), new=16):
     """Pazivik beside Zatusun at equal width and number of layer runs."""
     from .modeling_pazivik import PazivikConfig, PazivikForCausalLM
@@ -404,7 +468,7 @@ def run(pk, widths=(2048, 4096), n_layers=8, prompt=2048, decode_ctx=2048, decod
         m = DavasunForCausalLM(cfg, dev, BF16).init_weights(seed=1)
         d = step_model(m, cfg, pk, g, prompt, decode_ctx, decode_batches, new)
         rec["davasun"] = d
-        del eng, m
+        del m
         torch.cuda.empty_cache()
         # ---------------- OPT at equal width and depth (head_dim 128, 4x feed-forward)
         ocfg = OPTConfig(hidden_size=width, num_hidden_layers=n_layers, num_attention_heads=width // 128, ffn_dim=4 * width,

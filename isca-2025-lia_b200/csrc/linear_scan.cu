@@ -24,10 +24,10 @@
 //
 // Two more recurrences, on inputs that conv_act has made fp32:
 //   ssd_scan    (state-space duality, a scalar decay per head and token):   S_t = g_t S_{t-1} + dt_t B_t x_t^T,   y_t = S_t^T C_t + D_h x_t.
-//               State [vdim][N] per (slot, head) as above, but lanes share columns: a thread owns N / 8 rows of two columns, so one 128-bit
-//               read of B or C serves 8 cells and a token's two sums meet in three exchanges.
+//               State [vdim][N] per (slot, head) as above, but lanes share columns: a thread owns N / 16 rows of four columns, so one 128-bit
+//               read of B or C serves 16 cells, and the sums of several tokens meet in one round of exchanges.
 //   rglru_scan  (real-gated linear recurrent unit, one number per channel): S_t = a_t S_{t-1} + sqrt(1 - a_t^2) i_t u_t,  out_t = S_t gelu(y_t).
-//               64 tokens at a time: 16 warps fold 4 tokens each into one affine map, the maps are chained through shared memory.
+//               128 tokens at a time: 32 half-warps fold 4 tokens each into one affine map, the maps are chained through shared memory.
 #include <math.h>
 
 #include "common.cuh"
@@ -438,6 +438,9 @@ struct ConvActArgs {
   int dt_col, H;
 };
 
+constexpr int CONV_STRIP = 8;
+
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 __device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z))); }
 
 template <typename T, int TM>
@@ -467,6 +470,24 @@ __global__ void __launch_bounds__(256) conv_act_kernel(const T* __restrict__ y, 
     w[j] = j < a.taps ? wconv[(size_t)c * a.taps + a.taps - 1 - j] : 0.f;
     win[j] = 0.f;
   }
+  if (r1 - r0 == CONV_STRIP && r0 >= TM - 1) {
+    // a whole strip in the middle of a portion: all its inputs are rows of y, fetched together
+    const int slot = meta[2 * r0], pos = meta[2 * r0 + 1];
+    if (meta[2 * (r1 - 1)] == slot && meta[2 * (r1 - 1) + 1] == pos + CONV_STRIP - 1 && meta[2 * (r0 - TM + 1)] == slot && meta[2 * (r0 - TM + 1) + 1] == pos - TM + 1) {
+      float in[CONV_STRIP + TM - 1];
+#pragma unroll
+      for (int i = 0; i < CONV_STRIP + TM - 1; ++i) in[i] = ldf(col + (size_t)(r0 - TM + 1 + i) * a.ld);
+#pragma unroll
+      for (int i = 0; i < CONV_STRIP; ++i) {
+        float acc = ob;
+#pragma unroll
+        for (int j = 0; j < TM; ++j) acc = fmaf(w[j], in[i + TM - 1 - j] + ib, acc);       // (weights beyond the taps are zero)
+        if (a.act == LIA_ACT_SILU) acc = silu_fast(acc);
+        out[(size_t)(r0 + i) * a.ldo + c] = acc;
+      }
+      return;
+    }
+  }
   int pslot = -1, ppos = -1;
   for (int r = r0; r < r1; ++r) {
     const int slot = meta[2 * r], pos = meta[2 * r + 1];
@@ -490,7 +511,7 @@ __global__ void __launch_bounds__(256) conv_act_kernel(const T* __restrict__ y, 
     for (int j = 0; j < TM; ++j)
       if (j < a.taps && j <= pos) acc = fmaf(w[j], win[j] + ib, acc);
     acc += ob;
-    if (a.act == LIA_ACT_SILU) acc = silu(acc);
+    if (a.act == LIA_ACT_SILU) acc = silu_fast(acc);
     out[(size_t)r * a.ldo + c] = acc;
     if (a.single) {
 #pragma unroll
@@ -512,32 +533,33 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-constexpr int SSD_TB = 8;         // tokens per stage
-constexpr int SSD_COLS = 32;      // columns (of vdim) per block: 4 warps x 8
+constexpr int SSD_TB = 16;        // tokens per stage
 
-// Block: 32 columns of one head of one portion.  Lane: row group rg = lane & 7 owns rows 32 j + 4 rg .. + 3 (j < NJ, N <= 32 NJ), column
-// group lane >> 3 owns two columns.  Stages of SSD_TB tokens (B | C | x of this block's columns | dt | g) arrive by cp.async one stage ahead.
-template <int NJ, bool VL>
-__global__ void __launch_bounds__(128) ssd_scan_kernel(const float* __restrict__ B, const float* __restrict__ C, const float* __restrict__ x, int ld,
+// Block: 4 warps x 4 * 32 / RG columns of one head of one portion.  Lane: row group rg = lane % RG owns rows 4 RG j + 4 rg .. + 3 (j < NJ, N <= 4 RG NJ)
+// of the four columns of column group lane / RG.  TG tokens exchange their sums together (the unrolled body of TG tokens must stay small
+// enough for the instruction cache: there is one warp per scheduler to hide a miss).  Stages of SSD_TB tokens (B | C | x of this block's columns | dt | g) arrive by cp.async
+// one stage ahead.
+template <int NJ, int RG, int TG, bool VL>
+__global__ void __launch_bounds__(128, 1) ssd_scan_kernel(const float* __restrict__ B, const float* __restrict__ C, const float* __restrict__ x, int ld,
                                                        const float* __restrict__ gates, const float* __restrict__ D, float* __restrict__ St,
                                                        const int* __restrict__ segs, int H, int G, int N, int vdim, float* __restrict__ o) {
-  constexpr int NP = NJ * 32, ROWF = 2 * NP + SSD_COLS + 4;
+  constexpr int SSD_COLS = 4 * 4 * 32 / RG, NP = NJ * 4 * RG, ROWF = 2 * NP + SSD_COLS + 4;
   extern __shared__ __align__(16) float stage[];       // [2][SSD_TB][ROWF]
   const int seg = blockIdx.z, h = blockIdx.y, colb = blockIdx.x * SSD_COLS, g = h / (H / G);
   const int slot = segs[4 * seg], row0 = segs[4 * seg + 2], len = segs[4 * seg + 3];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7;
-  const int cl = warp * 8 + (lane >> 3) * 2, col0 = colb + cl;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane % RG;
+  const int cl = warp * (SSD_COLS / 4) + (lane / RG) * 4, col0 = colb + cl;
   const int ncol = min(SSD_COLS, vdim - colb);
 
   for (int i = threadIdx.x; i < 2 * SSD_TB * ROWF; i += 128) stage[i] = 0.f;      // rows N .. NP-1 of B and C stay zero
-  float S[2][NJ * 4];
+  float S[4][NJ * 4];
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < 4; ++c) {
     const float* Sp = St + (((size_t)slot * H + h) * vdim + col0 + c) * N;
     const bool live = col0 + c < vdim;
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-      const int r = 32 * j + 4 * rg;
+      const int r = 4 * RG * j + 4 * rg;
       if (VL) {
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         if (live && r < N) v = *reinterpret_cast<const float4*>(Sp + r);
@@ -551,25 +573,75 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const float* __restrict__
   __syncthreads();
 
   constexpr int U = VL ? 4 : 1;                        // floats per copy
-  const int n_u = N / U, x_u = VL ? ncol / 4 : ncol, per_tok = 2 * n_u + x_u;
+  constexpr int SLOTS = (SSD_TB * (2 * NP + SSD_COLS) / 4 + 127) / 128;            // copies of 4 floats per thread and stage
+  const int n_u = N / U, x_u = ncol / U, per_tok = 2 * n_u + x_u;
+  // copy e of a stage: token e / per_tok, then B | C | x in order
+  auto place = [&](int e, int& t, size_t& src, int& which, int& dst) {
+    t = e / per_tok;
+    const int j = e - t * per_tok;
+    which = j < n_u ? 0 : (j < 2 * n_u ? 1 : 2);
+    const int k = (j - which * n_u) * U;
+    src = (size_t)(row0 + t) * ld + (which == 2 ? h * vdim + colb : g * N) + k;
+    dst = t * ROWF + which * NP + k;
+  };
+  const float* slot_src[VL ? SLOTS : 1];               // the copies of this thread, moved on stage by stage
+  int slot_dst[VL ? SLOTS : 1];
+  if constexpr (VL) {
+#pragma unroll
+    for (int i = 0; i < SLOTS; ++i) {
+      int t, which;
+      size_t src;
+      place(threadIdx.x + i * 128, t, src, which, slot_dst[i]);
+      slot_src[i] = (which == 0 ? B : (which == 1 ? C : x)) + src;
+      if (t >= SSD_TB) slot_dst[i] = -1;
+    }
+  }
   auto fetch = [&](int gidx) {
     const int t0 = gidx * SSD_TB, nt = min(SSD_TB, len - t0);
     float* st = stage + (gidx & 1) * SSD_TB * ROWF;
-    for (int e = threadIdx.x; e < nt * per_tok; e += 128) {
-      const int t = e / per_tok, j = e - t * per_tok;
-      const size_t row = (size_t)(row0 + t0 + t) * ld;
-      const float* src;
-      float* dst = st + t * ROWF;
-      if (j < n_u) { src = B + row + g * N + j * U; dst += j * U; }
-      else if (j < 2 * n_u) { src = C + row + g * N + (j - n_u) * U; dst += NP + (j - n_u) * U; }
-      else { src = x + row + (size_t)h * vdim + colb + (j - 2 * n_u) * U; dst += 2 * NP + (j - 2 * n_u) * U; }
-      if (VL) cp_async16(dst, src);
-      else cp_async4(dst, src);
+    if constexpr (VL) {
+#pragma unroll
+      for (int i = 0; i < SLOTS; ++i) {
+        if (slot_dst[i] >= 0 && slot_dst[i] < nt * ROWF) cp_async16(st + slot_dst[i], slot_src[i]);
+        slot_src[i] += (size_t)SSD_TB * ld;
+      }
+    } else {
+      for (int e = threadIdx.x; e < nt * per_tok; e += 128) {
+        int t, which, dst;
+        size_t src;
+        place(e, t, src, which, dst);
+        cp_async4(st + dst, (which == 0 ? B : (which == 1 ? C : x)) + src + (size_t)t0 * ld);
+      }
     }
     if (threadIdx.x < 2 * nt) {
       const int t = threadIdx.x >> 1, which = threadIdx.x & 1;
       cp_async4(st + t * ROWF + 2 * NP + SSD_COLS + which, gates + (size_t)(row0 + t0 + t) * 2 * H + which * H + h);
     }
+  };
+  // one token: the state moves on; s = this thread's part of the four columns' sums
+  auto token = [&](const float* tk, float4 xv, float* s) {
+    const float2 dg = *reinterpret_cast<const float2*>(tk + 2 * NP + SSD_COLS);
+    const float u[4] = {dg.x * xv.x, dg.x * xv.y, dg.x * xv.z, dg.x * xv.w};
+    float hi[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) s[c] = hi[c] = 0.f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const float4 k = *reinterpret_cast<const float4*>(tk + 4 * RG * j + 4 * rg);
+      const float4 q = *reinterpret_cast<const float4*>(tk + NP + 4 * RG * j + 4 * rg);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float* Sc = S[c] + 4 * j;
+        Sc[0] = fmaf(dg.y, Sc[0], k.x * u[c]);
+        Sc[1] = fmaf(dg.y, Sc[1], k.y * u[c]);
+        Sc[2] = fmaf(dg.y, Sc[2], k.z * u[c]);
+        Sc[3] = fmaf(dg.y, Sc[3], k.w * u[c]);
+        s[c] = fmaf(Sc[1], q.y, fmaf(Sc[0], q.x, s[c]));
+        hi[c] = fmaf(Sc[3], q.w, fmaf(Sc[2], q.z, hi[c]));
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c) s[c] += hi[c];
   };
   const float dh = D[h];
   const int groups = (len + SSD_TB - 1) / SSD_TB;
@@ -583,52 +655,53 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const float* __restrict__
     const float* st = stage + (gi & 1) * SSD_TB * ROWF;
     const int nt = min(SSD_TB, len - gi * SSD_TB);
     float* orow = o + (size_t)(row0 + gi * SSD_TB) * H * vdim + (size_t)h * vdim + colb;
-#pragma unroll 2
-    for (int t = 0; t < nt; ++t) {
-      const float* tk = st + t * ROWF;
-      const float2 xv = *reinterpret_cast<const float2*>(tk + 2 * NP + cl);
-      const float2 dg = *reinterpret_cast<const float2*>(tk + 2 * NP + SSD_COLS);
-      const float u0 = dg.x * xv.x, u1 = dg.x * xv.y;
-      float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
+    // lane rg ends with the sums e, e + 1, .. of n: every exchange of the loop halves what a lane holds until one is left
+    auto exchange = [&](float* s, int n) {
 #pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        const float4 k = *reinterpret_cast<const float4*>(tk + 32 * j + 4 * rg);
-        const float4 q = *reinterpret_cast<const float4*>(tk + NP + 32 * j + 4 * rg);
-        S[0][4 * j] = fmaf(dg.y, S[0][4 * j], k.x * u0);
-        S[1][4 * j] = fmaf(dg.y, S[1][4 * j], k.x * u1);
-        a0 = fmaf(S[0][4 * j], q.x, a0);
-        a1 = fmaf(S[1][4 * j], q.x, a1);
-        S[0][4 * j + 1] = fmaf(dg.y, S[0][4 * j + 1], k.y * u0);
-        S[1][4 * j + 1] = fmaf(dg.y, S[1][4 * j + 1], k.y * u1);
-        b0 = fmaf(S[0][4 * j + 1], q.y, b0);
-        b1 = fmaf(S[1][4 * j + 1], q.y, b1);
-        S[0][4 * j + 2] = fmaf(dg.y, S[0][4 * j + 2], k.z * u0);
-        S[1][4 * j + 2] = fmaf(dg.y, S[1][4 * j + 2], k.z * u1);
-        a0 = fmaf(S[0][4 * j + 2], q.z, a0);
-        a1 = fmaf(S[1][4 * j + 2], q.z, a1);
-        S[0][4 * j + 3] = fmaf(dg.y, S[0][4 * j + 3], k.w * u0);
-        S[1][4 * j + 3] = fmaf(dg.y, S[1][4 * j + 3], k.w * u1);
-        b0 = fmaf(S[0][4 * j + 3], q.w, b0);
-        b1 = fmaf(S[1][4 * j + 3], q.w, b1);
+      for (int w = RG / 2; w > 0; w >>= 1) {
+        n >>= 1;
+        const bool up = rg & w;
+#pragma unroll
+        for (int i = 0; i < n; ++i) {
+          const float keep = up ? s[i + n] : s[i], give = up ? s[i] : s[i + n];
+          s[i] = keep + __shfl_xor_sync(0xffffffffu, give, w);
+        }
+        if (n == 0) s[0] += __shfl_xor_sync(0xffffffffu, s[0], w);
       }
-      a0 += b0;
-      a1 += b1;
-      // even row groups go on with column 0, odd ones with column 1
-      const bool odd = rg & 1;
-      float sum = (odd ? a1 : a0) + __shfl_xor_sync(0xffffffffu, odd ? a0 : a1, 1);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-      sum += __shfl_xor_sync(0xffffffffu, sum, 4);
-      if (rg < 2 && cl + rg < ncol) orow[(size_t)t * H * vdim + cl + rg] = fmaf(dh, odd ? xv.y : xv.x, sum);
+    };
+    auto put = [&](int t, int c, float sum) {
+      if (c < ncol) orow[(size_t)t * H * vdim + c] = fmaf(dh, st[t * ROWF + 2 * NP + c], sum);
+    };
+    int t0 = 0;
+#pragma unroll 1
+    for (; t0 + TG <= nt; t0 += TG) {
+      float s[TG * 4];
+#pragma unroll
+      for (int t = 0; t < TG; ++t) token(st + (t0 + t) * ROWF, *reinterpret_cast<const float4*>(st + (t0 + t) * ROWF + 2 * NP + cl), s + 4 * t);
+      exchange(s, TG * 4);
+      constexpr int PER = TG * 4 / RG > 0 ? TG * 4 / RG : 1, REP = RG / (TG * 4) > 0 ? RG / (TG * 4) : 1;     // sums per lane, lanes per sum
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int e = rg / REP * PER + i;
+        if (rg % REP == 0) put(t0 + e / 4, cl + e % 4, s[i]);
+      }
+    }
+#pragma unroll 1
+    for (; t0 < nt; ++t0) {
+      float s[4];
+      token(st + t0 * ROWF, *reinterpret_cast<const float4*>(st + t0 * ROWF + 2 * NP + cl), s);
+      exchange(s, 4);
+      if (rg % (RG / 4) == 0) put(t0, cl + rg / (RG / 4), s[0]);
     }
     __syncthreads();                                   // the stage after next goes where this one was
   }
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < 4; ++c) {
     if (col0 + c >= vdim) continue;
     float* Sp = St + (((size_t)slot * H + h) * vdim + col0 + c) * N;
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
-      const int r = 32 * j + 4 * rg;
+      const int r = 4 * RG * j + 4 * rg;
       if (VL) {
         if (r < N) *reinterpret_cast<float4*>(Sp + r) = make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]);
       } else {
@@ -640,39 +713,45 @@ __global__ void __launch_bounds__(128) ssd_scan_kernel(const float* __restrict__
   }
 }
 
-template <int NJ, bool VL>
+template <int NJ, int RG, int TG, bool VL>
 int launch_ssd_as(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs, int nseg, int H,
                   int G, int N, int vdim, float* o, cudaStream_t stream) {
-  const size_t smem = (size_t)2 * SSD_TB * (2 * NJ * 32 + SSD_COLS + 4) * sizeof(float);
-  if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(ssd_scan_kernel<NJ, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  dim3 grid((vdim + SSD_COLS - 1) / SSD_COLS, H, nseg);
-  ssd_scan_kernel<NJ, VL><<<grid, 128, smem, stream>>>(B, C, x, ld, gates, D, St, segs, H, G, N, vdim, o);
+  constexpr int COLS = 16 * 32 / RG;
+  const size_t smem = (size_t)2 * SSD_TB * (2 * NJ * 4 * RG + COLS + 4) * sizeof(float);
+  if (smem > 48 * 1024) LIA_CUDA(cudaFuncSetAttribute(ssd_scan_kernel<NJ, RG, TG, VL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  dim3 grid((vdim + COLS - 1) / COLS, H, nseg);
+  ssd_scan_kernel<NJ, RG, TG, VL><<<grid, 128, smem, stream>>>(B, C, x, ld, gates, D, St, segs, H, G, N, vdim, o);
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }
 
 // 128-bit copies and state accesses: every B, C, x segment and every state column starts on a 16-byte boundary
-template <int NJ>
+template <int NJ, int RG, int TG>
 int launch_ssd(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs, int nseg, int H,
                int G, int N, int vdim, float* o, cudaStream_t stream) {
   const bool aligned = ((reinterpret_cast<uintptr_t>(B) | reinterpret_cast<uintptr_t>(C) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(St)) % 16 == 0) &&
                        ld % 4 == 0 && N % 4 == 0 && vdim % 4 == 0;
-  if (aligned) return launch_ssd_as<NJ, true>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
-  return launch_ssd_as<NJ, false>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
+  if (aligned) return launch_ssd_as<NJ, RG, TG, true>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
+  return launch_ssd_as<NJ, RG, TG, false>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------- gated linear recurrent unit
-constexpr int LRU_W = 16, LRU_T = 4;          // warps per block, tokens per warp and sweep
+constexpr int LRU_W = 16, LRU_T = 4, LRU_CH = 16;          // warps per block, tokens per thread and sweep, channels per block
 
-// Block: 32 channels of one portion.  z [rows][blocks][2 n] holds every channel block's gate projections r | i (n = width / blocks),
-// z_bias [blocks][2 n] their biases, c[ch] = -8 softplus(lam): log a = c sigmoid(r).
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
+
+// Block: 16 channels of one portion; a half-warp takes LRU_T consecutive tokens of a sweep.  z [rows][blocks][2 n] holds every channel block's gate
+// projections r | i (n = width / blocks), z_bias [blocks][2 n] their biases, c[ch] = -8 softplus(lam): log a = c sigmoid(r).
 template <typename T>
 __global__ void __launch_bounds__(LRU_W * 32) rglru_scan_kernel(const float* __restrict__ u, const float* __restrict__ z, const float* __restrict__ z_bias,
                                                                 const float* __restrict__ c, const T* __restrict__ y, int ldy, const float* __restrict__ y_bias,
                                                                 float* __restrict__ St, const int* __restrict__ segs, int width, int n, T* __restrict__ out) {
-  __shared__ float2 maps[2][LRU_W][32];       // a warp's four tokens as S -> x S + y
+  constexpr int SWEEP = LRU_W * 2 * LRU_T;
+  __shared__ float2 maps[2][LRU_W][LRU_CH];   // a warp's eight tokens as S -> x S + y
   const int seg = blockIdx.y, slot = segs[4 * seg], row0 = segs[4 * seg + 2], len = segs[4 * seg + 3];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ch = blockIdx.x * 32 + lane;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, cl = lane & (LRU_CH - 1), ch = blockIdx.x * LRU_CH + cl;
+  const bool upper = lane >= LRU_CH;
+  const int first = (threadIdx.x / LRU_CH) * LRU_T;
   const bool live = ch < width;
   const int blk = live ? ch / n : 0, zc = blk * 2 * n + (live ? ch - blk * n : 0);
   const float cc = live ? c[ch] : 0.f, rb = live ? z_bias[zc] : 0.f, ib = live ? z_bias[zc + n] : 0.f, yb = (live && y_bias) ? y_bias[ch] : 0.f;
@@ -681,7 +760,7 @@ __global__ void __launch_bounds__(LRU_W * 32) rglru_scan_kernel(const float* __r
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < LRU_T; ++k) {
-      const int t = t0 + warp * LRU_T + k;
+      const int t = t0 + first + k;
       ur[k] = zr[k] = zi[k] = yr[k] = 0.f;
       if (live && t < len) {
         const size_t row = (size_t)(row0 + t);
@@ -694,40 +773,42 @@ __global__ void __launch_bounds__(LRU_W * 32) rglru_scan_kernel(const float* __r
   };
   fetch(0);
   int buf = 0;
-  for (int t0 = 0; t0 < len; t0 += LRU_W * LRU_T) {
+  for (int t0 = 0; t0 < len; t0 += SWEEP) {
     float a[LRU_T], b[LRU_T], g[LRU_T], pa = 1.f, pb = 0.f;
 #pragma unroll
     for (int k = 0; k < LRU_T; ++k) {
       a[k] = 1.f;
       b[k] = g[k] = 0.f;
-      if (t0 + warp * LRU_T + k < len) {
-        const float la = cc / (1.0f + expf(-(zr[k] + rb)));
+      if (t0 + first + k < len) {
+        const float la = cc * sigmoid_fast(zr[k] + rb);
         a[k] = expf(la);
-        b[k] = sqrtf(-expm1f(2.0f * la)) * ur[k] / (1.0f + expf(-(zi[k] + ib)));
+        b[k] = sqrtf(-expm1f(2.0f * la)) * ur[k] * sigmoid_fast(zi[k] + ib);
         g[k] = gelu_tanh(yr[k] + yb);
       }
       pa *= a[k];
       pb = fmaf(a[k], pb, b[k]);
     }
-    maps[buf][warp][lane] = make_float2(pa, pb);
-    if (t0 + LRU_W * LRU_T < len) fetch(t0 + LRU_W * LRU_T);
+    const float la = __shfl_sync(0xffffffffu, pa, cl), lb = __shfl_sync(0xffffffffu, pb, cl);      // the lower half's map
+    if (upper) maps[buf][warp][cl] = make_float2(pa * la, fmaf(pa, lb, pb));
+    if (t0 + SWEEP < len) fetch(t0 + SWEEP);
     __syncthreads();
     float s = S;
 #pragma unroll
     for (int w = 0; w < LRU_W; ++w) {
       if (w == warp) s = S;
-      const float2 m = maps[buf][w][lane];
+      const float2 m = maps[buf][w][cl];
       S = fmaf(m.x, S, m.y);
     }
+    if (upper) s = fmaf(la, s, lb);
 #pragma unroll
     for (int k = 0; k < LRU_T; ++k) {
-      const int t = t0 + warp * LRU_T + k;
+      const int t = t0 + first + k;
       s = fmaf(a[k], s, b[k]);
       if (live && t < len) out[(size_t)(row0 + t) * width + ch] = T(s * g[k]);
     }
     buf ^= 1;                                 // the other half: last read before the barrier above
   }
-  if (warp == 0 && live) St[(size_t)slot * width + ch] = S;
+  if (threadIdx.x < LRU_CH && live) St[(size_t)slot * width + ch] = S;
 }
 
 }  // namespace
@@ -811,7 +892,7 @@ extern "C" int lia_conv_act(const void* y, int y_f32, int ld, int col0, int C, c
   LIA_CHECK_ARG(act == LIA_ACT_NONE || act == LIA_ACT_SILU, "lia_conv_act: unknown activation %d", act);
   LIA_CHECK_ARG(H >= 0 && (H == 0 || (dt_bias && a_log && gates && dt_col >= 0 && ld >= dt_col + H)), "lia_conv_act: bad step sizes (H=%d)", H);
   const int single = nseg == M && taps > 1;      // every portion is one row
-  ConvActArgs a{ld, col0, C, taps, act, single, ldo, M, M <= 64 ? 1 : 8, dt_col, H};
+  ConvActArgs a{ld, col0, C, taps, act, single, ldo, M, M <= 64 ? 1 : CONV_STRIP, dt_col, H};
   dim3 grid((C + H + 255) / 256, (M + a.strip - 1) / a.strip);
   LIA_CHECK_ARG(grid.y <= 65535, "lia_conv_act: too many rows (%d)", M);
 #define LIA_CA(T, TM) conv_act_kernel<T, TM><<<grid, 256, 0, stream>>>(reinterpret_cast<const T*>(y), in_bias, wconv, bias, state, meta, out, dt_bias, a_log, gates, a)
@@ -840,11 +921,10 @@ extern "C" int lia_ssd_scan(const float* B, const float* C, const float* x, int 
   LIA_CHECK_ARG(B && C && x && gates && D && state_S && segs && o, "lia_ssd_scan: null pointer");
   LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && N > 0 && N <= 512 && vdim > 0,
                 "lia_ssd_scan: bad shape nseg=%d H=%d G=%d N=%d vdim=%d", nseg, H, G, N, vdim);
-  if (N <= 32) return launch_ssd<1>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  if (N <= 64) return launch_ssd<2>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  if (N <= 128) return launch_ssd<4>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  if (N <= 256) return launch_ssd<8>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  return launch_ssd<16>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 64) return launch_ssd<1, 16, 8>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 128) return launch_ssd<2, 16, 4>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 256) return launch_ssd<4, 16, 2>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  return launch_ssd<8, 16, 1>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
 }
 
 extern "C" int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
@@ -852,7 +932,7 @@ extern "C" int lia_rglru_scan(const float* u, const float* z, const float* z_bia
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(u && z && z_bias && c && y && state && segs && out, "lia_rglru_scan: null pointer");
   LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && width > 0 && blocks > 0 && width % blocks == 0 && ldy >= width, "lia_rglru_scan: bad shape width=%d blocks=%d", width, blocks);
-  dim3 grid((width + 31) / 32, nseg);
+  dim3 grid((width + LRU_CH - 1) / LRU_CH, nseg);
   if (y_f32) rglru_scan_kernel<float><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const float*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<float*>(out));
   else rglru_scan_kernel<bf16><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const bf16*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<bf16*>(out));
   LIA_LAUNCH_CHECK();
