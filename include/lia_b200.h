@@ -548,14 +548,15 @@ int lia_conv_act(const void* y, int y_f32, int ld, int col0, int C, const float*
                  float* state, const int* meta, const int* segs, int nseg, float* out, int ldo, int M, int dt_col, int H, const float* dt_bias,
                  const float* a_log, float* gates, lia_stream_t stream);
 /* State-space dual recurrence over every portion, per head h (B and C of group h / (H / G), N <= 512 numbers; x of vdim numbers; all with
- * row stride ld):  S = g S + dt B x^T,  o = S^T C + D[h] x;  gates [rows][2H] = dt | g; state_S [slot][H][vdim][N], o [rows][H * vdim] fp32 */
+ * row stride ld):  S = g S + dt B x^T,  o = S^T C + D[h] x;  gates [rows][2H] = dt | g; state_S [slot][H][vdim][N], o [rows][H * vdim] fp32;
+ * rows: tokens of all nseg portions together */
 int lia_ssd_scan(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* state_S, const int* segs, int nseg,
-                 int H, int G, int N, int vdim, float* o, lia_stream_t stream);
+                 int rows, int H, int G, int N, int vdim, float* o, lia_stream_t stream);
 /* Real-gated linear recurrent unit over every portion, channel by channel (width = blocks * n): log a = c sigmoid(r + its bias),
  * S = a S + sqrt(1 - a^2) sigmoid(i + its bias) u, out = S * gelu_tanh(y + y_bias) of y's type; z [rows][blocks][2n] = r | i,
- * z_bias [blocks][2n], state [slot][width] fp32; y has row stride ldy, y_bias may be NULL */
+ * z_bias [blocks][2n], state [slot][width] fp32; y has row stride ldy, y_bias may be NULL; rows as above */
 int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
-                   float* state, const int* segs, int nseg, int width, int blocks, void* out, lia_stream_t stream);
+                   float* state, const int* segs, int nseg, int rows, int width, int blocks, void* out, lia_stream_t stream);
 /* lia_router_topk_scored with groups > 1: the experts form that many equal groups of neighbours, a group ranks by its largest choice score
  * and only experts of the `keep` best groups can be chosen (top <= keep * E / groups) */
 int lia_router_topk_grouped(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int groups, int keep, int* idx,

@@ -540,7 +540,7 @@ constexpr int SSD_TB = 16;        // tokens per stage
 // enough for the instruction cache: there is one warp per scheduler to hide a miss).  Stages of SSD_TB tokens (B | C | x of this block's columns | dt | g) arrive by cp.async
 // one stage ahead.
 template <int NJ, int RG, int TG, bool VL>
-__global__ void __launch_bounds__(128, 1) ssd_scan_kernel(const float* __restrict__ B, const float* __restrict__ C, const float* __restrict__ x, int ld,
+__global__ void __launch_bounds__(128, TG > 1 ? 1 : (NJ <= 2 ? 5 : (NJ <= 4 ? 3 : 1))) ssd_scan_kernel(const float* __restrict__ B, const float* __restrict__ C, const float* __restrict__ x, int ld,
                                                        const float* __restrict__ gates, const float* __restrict__ D, float* __restrict__ St,
                                                        const int* __restrict__ segs, int H, int G, int N, int vdim, float* __restrict__ o) {
   constexpr int SSD_COLS = 4 * 4 * 32 / RG, NP = NJ * 4 * RG, ROWF = 2 * NP + SSD_COLS + 4;
@@ -551,7 +551,8 @@ __global__ void __launch_bounds__(128, 1) ssd_scan_kernel(const float* __restric
   const int cl = warp * (SSD_COLS / 4) + (lane / RG) * 4, col0 = colb + cl;
   const int ncol = min(SSD_COLS, vdim - colb);
 
-  for (int i = threadIdx.x; i < 2 * SSD_TB * ROWF; i += 128) stage[i] = 0.f;      // rows N .. NP-1 of B and C stay zero
+  if (N < NP || ncol < SSD_COLS)                       // rows N .. NP-1 of B and C and the columns beyond vdim stay zero
+    for (int i = threadIdx.x; i < min(2 * SSD_TB, len) * ROWF; i += 128) stage[i] = 0.f;
   float S[4][NJ * 4];
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
@@ -726,23 +727,25 @@ int launch_ssd_as(const float* B, const float* C, const float* x, int ld, const 
 }
 
 // 128-bit copies and state accesses: every B, C, x segment and every state column starts on a 16-byte boundary
+// single: every portion is one token (decoding) -- the variant without token groups needs fewer registers, so more blocks share an SM
 template <int NJ, int RG, int TG>
-int launch_ssd(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs, int nseg, int H,
-               int G, int N, int vdim, float* o, cudaStream_t stream) {
+int launch_ssd(bool single, const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* St, const int* segs,
+               int nseg, int H, int G, int N, int vdim, float* o, cudaStream_t stream) {
   const bool aligned = ((reinterpret_cast<uintptr_t>(B) | reinterpret_cast<uintptr_t>(C) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(St)) % 16 == 0) &&
                        ld % 4 == 0 && N % 4 == 0 && vdim % 4 == 0;
+  if (aligned && single) return launch_ssd_as<NJ, RG, 1, true>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
   if (aligned) return launch_ssd_as<NJ, RG, TG, true>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
   return launch_ssd_as<NJ, RG, TG, false>(B, C, x, ld, gates, D, St, segs, nseg, H, G, N, vdim, o, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------- gated linear recurrent unit
-constexpr int LRU_W = 16, LRU_T = 4, LRU_CH = 16;          // warps per block, tokens per thread and sweep, channels per block
+constexpr int LRU_T = 4, LRU_CH = 16;          // tokens per thread and sweep, channels per block
 
 __device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 
-// Block: 16 channels of one portion; a half-warp takes LRU_T consecutive tokens of a sweep.  z [rows][blocks][2 n] holds every channel block's gate
+// Block: 16 channels of one portion, LRU_W warps (16; 1 in a step of single tokens); a half-warp takes LRU_T consecutive tokens of a sweep.  z [rows][blocks][2 n] holds every channel block's gate
 // projections r | i (n = width / blocks), z_bias [blocks][2 n] their biases, c[ch] = -8 softplus(lam): log a = c sigmoid(r).
-template <typename T>
+template <typename T, int LRU_W>
 __global__ void __launch_bounds__(LRU_W * 32) rglru_scan_kernel(const float* __restrict__ u, const float* __restrict__ z, const float* __restrict__ z_bias,
                                                                 const float* __restrict__ c, const T* __restrict__ y, int ldy, const float* __restrict__ y_bias,
                                                                 float* __restrict__ St, const int* __restrict__ segs, int width, int n, T* __restrict__ out) {
@@ -916,25 +919,31 @@ extern "C" int lia_conv_act(const void* y, int y_f32, int ld, int col0, int C, c
 }
 
 extern "C" int lia_ssd_scan(const float* B, const float* C, const float* x, int ld, const float* gates, const float* D, float* state_S, const int* segs,
-                            int nseg, int H, int G, int N, int vdim, float* o, lia_stream_t stream_) {
+                            int nseg, int rows, int H, int G, int N, int vdim, float* o, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  const bool single = rows == nseg;
+  LIA_CHECK_ARG(rows >= nseg, "lia_ssd_scan: fewer rows (%d) than portions (%d)", rows, nseg);
   LIA_CHECK_ARG(B && C && x && gates && D && state_S && segs && o, "lia_ssd_scan: null pointer");
   LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && N > 0 && N <= 512 && vdim > 0,
                 "lia_ssd_scan: bad shape nseg=%d H=%d G=%d N=%d vdim=%d", nseg, H, G, N, vdim);
-  if (N <= 64) return launch_ssd<1, 16, 8>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  if (N <= 128) return launch_ssd<2, 16, 4>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  if (N <= 256) return launch_ssd<4, 16, 2>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
-  return launch_ssd<8, 16, 1>(B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 64) return launch_ssd<1, 16, 8>(single, B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 128) return launch_ssd<2, 16, 4>(single, B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  if (N <= 256) return launch_ssd<4, 16, 2>(single, B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
+  return launch_ssd<8, 16, 1>(single, B, C, x, ld, gates, D, state_S, segs, nseg, H, G, N, vdim, o, stream);
 }
 
 extern "C" int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
-                              float* state, const int* segs, int nseg, int width, int blocks, void* out, lia_stream_t stream_) {
+                              float* state, const int* segs, int nseg, int rows, int width, int blocks, void* out, lia_stream_t stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   LIA_CHECK_ARG(u && z && z_bias && c && y && state && segs && out, "lia_rglru_scan: null pointer");
-  LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && width > 0 && blocks > 0 && width % blocks == 0 && ldy >= width, "lia_rglru_scan: bad shape width=%d blocks=%d", width, blocks);
+  LIA_CHECK_ARG(nseg > 0 && nseg <= 65535 && rows >= nseg && width > 0 && blocks > 0 && width % blocks == 0 && ldy >= width, "lia_rglru_scan: bad shape width=%d blocks=%d", width, blocks);
   dim3 grid((width + LRU_CH - 1) / LRU_CH, nseg);
-  if (y_f32) rglru_scan_kernel<float><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const float*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<float*>(out));
-  else rglru_scan_kernel<bf16><<<grid, LRU_W * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const bf16*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<bf16*>(out));
+#define LIA_RS(T, W_) rglru_scan_kernel<T, W_><<<grid, W_ * 32, 0, stream>>>(u, z, z_bias, c, reinterpret_cast<const T*>(y), ldy, y_bias, state, segs, width, width / blocks, reinterpret_cast<T*>(out))
+  if (y_f32 && rows == nseg) LIA_RS(float, 1);
+  else if (y_f32) LIA_RS(float, 16);
+  else if (rows == nseg) LIA_RS(bf16, 1);
+  else LIA_RS(bf16, 16);
+#undef LIA_RS
   LIA_LAUNCH_CHECK();
   return LIA_OK;
 }

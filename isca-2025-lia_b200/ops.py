@@ -1129,7 +1129,7 @@ def ssd_scan(xbc, gates, D, state_S, segs, H, G, N, vdim, o):
     if xbc.dtype != F32 or xbc.shape[1] != inner + 2 * G * N or tuple(gates.shape) != (M, 2 * H) or D.numel() != H or tuple(o.shape) != (M, inner) \
             or tuple(state_S.shape[1:]) != (H, vdim, N):
         raise _lib.LiaError("ssd_scan: shapes do not agree")
-    check(_lib.load().lia_ssd_scan(_p(xbc[:, inner:]), _p(xbc[:, inner + G * N:]), _p(xbc), ld, _p(gates), _p(D), _p(state_S), _p(segs), segs.shape[0], H, G, N,
+    check(_lib.load().lia_ssd_scan(_p(xbc[:, inner:]), _p(xbc[:, inner + G * N:]), _p(xbc), ld, _p(gates), _p(D), _p(state_S), _p(segs), segs.shape[0], M, H, G, N,
                                    vdim, _p(o), _stream()), "lia_ssd_scan")
     count_launches()
     return o
@@ -1148,7 +1148,7 @@ def rglru_scan(u, z, z_bias, c, y, y_bias, state, segs, blocks, out):
     if tuple(z.shape) != (M, 2 * width) or z_bias.numel() != 2 * width or c.numel() != width or tuple(y.shape) != (M, width) or tuple(state.shape[1:]) != (width,) \
             or width % blocks or not (out.is_cuda and out.is_contiguous() and tuple(out.shape) == (M, width) and out.dtype == y.dtype):
         raise _lib.LiaError("rglru_scan: shapes do not agree")
-    check(_lib.load().lia_rglru_scan(_p(u), _p(z), _p(z_bias), _p(c), _p(y), _f32(y), ldy, _p(y_bias), _p(state), _p(segs), segs.shape[0], width, int(blocks),
+    check(_lib.load().lia_rglru_scan(_p(u), _p(z), _p(z_bias), _p(c), _p(y), _f32(y), ldy, _p(y_bias), _p(state), _p(segs), segs.shape[0], M, width, int(blocks),
                                      _p(out), _stream()), "lia_rglru_scan")
     count_launches()
     return out
