@@ -557,8 +557,8 @@ int lia_ssd_scan(const float* B, const float* C, const float* x, int ld, const f
  * z_bias [blocks][2n], state [slot][width] fp32; y has row stride ldy, y_bias may be NULL; rows as above */
 int lia_rglru_scan(const float* u, const float* z, const float* z_bias, const float* c, const void* y, int y_f32, int ldy, const float* y_bias,
                    float* state, const int* segs, int nseg, int rows, int width, int blocks, void* out, lia_stream_t stream);
-/* lia_router_topk_scored with groups > 1: the experts form that many equal groups of neighbours, a group ranks by its largest choice score
- * and only experts of the `keep` best groups can be chosen (top <= keep * E / groups) */
+/* lia_router_topk_scored with groups > 1: the experts are cut into that many runs of E / groups; a run ranks by its largest choice score, and
+ * the choice is made inside the `keep` best runs (top <= keep * E / groups) */
 int lia_router_topk_grouped(const float* logits, int ldl, const float* correction, int renorm, int sigmoid, int groups, int keep, int* idx,
                             float* wt, int M, int E, int top, lia_stream_t stream);
 

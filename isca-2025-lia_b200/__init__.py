@@ -12,10 +12,12 @@ Layout:
   checkpoint.py    HF safetensors/.bin reader and the native per-layer slab format
   tp.py            tensor-parallel plumbing: peer arenas for the fused projection+all-reduce kernel, NCCL bootstrap
   run.py           the reference's run.py / run_generation.py command line
-  registry.py      config.json -> model class (OPT, Davasun, Bebulorn)
+  registry.py      config.json -> model class (OPT, Davasun, Bebulorn, Bizetar, Zatusun, Pazivik, Sekenex)
   modeling_davasun.py  Davasun: mLSTM + latent-attention layers on a 32-bit residual stream, looped layer block
   modeling_bebulorn.py Bebulorn: decay / delta-rule linear attention and sliding-window attention layers between layer norms,
                    dense or mixture-of-experts feed-forwards, looped layer block with the embedding added back
+  modeling_sekenex.py  Sekenex: state-space mixers and layers of attention beside a gated recurrent block on several residual streams
+                   (modeling_bizetar.py, modeling_zatusun.py, modeling_pazivik.py: the other step-served families)
   seq_layers.py    their mixers / feed-forward as general parts (constants are parameters); seq_state.py: per-request slots of
                    recurrent state and row caches; engine.py: the step function (requests, portions, mixed batches, greedy)
 """

@@ -1,7 +1,7 @@
 // Row operations of models that keep their residual stream in 32-bit floats: RMS norms with a scalar or a per-channel
 // weight (fused with the residual add that follows a sublayer and with the norm that precedes the next one), the token
 // embedding with its norm, with learned or wave positions and with a bigram table, the gated, normed residual update with a weighted mix of all earlier layers' results, the
-// residual kept as several streams that learned weights read, mix and write, a gate product behind a norm in groups, the
+// residual kept as several streams that learned weights read, mix and write, a gate product under a norm in groups, the
 // polynomial activation between norms, a gated feed-forward activation with clamps, a projection onto a handful of outputs with the
 // gate non-linearities in its epilogue, a plain strided-batched projection on the CUDA cores (true 32-bit products and
 // sums: the exact path, and the carrier of shapes the tensor-core GEMM does not take), and a 32-bit argmax.
@@ -444,8 +444,8 @@ __global__ void __launch_bounds__(256) streams_gather_kernel(const float* __rest
   for (int i = threadIdx.x; i < W; i += 256) stf(h + (size_t)blockIdx.x * W + i, us[i] * inv * w[i]);
 }
 
-// out = w * g / sqrt(mean(g^2) + eps), g = o * silu(z), the mean taken over each of `groups` equal parts of a row by itself (the gate comes
-// before the norm).  o fp32 [M][F], z of the activations' type with row stride ldz.  Block per (row, part); `us` keeps g (F / groups floats).
+// out = w * g / sqrt(mean(g^2) + eps), g = o * silu(z), the mean taken over each of `groups` equal parts of a row by itself (gated first,
+// normed second).  o fp32 [M][F], z of the activations' type with row stride ldz.  Block per (row, part); `us` keeps g (F / groups floats).
 template <typename T, int VEC>
 __global__ void __launch_bounds__(128) silu_gate_norm_kernel(const float* __restrict__ o, const T* __restrict__ z, int ldz, const float* __restrict__ w,
                                                              T* __restrict__ out, int F, int groups, float eps) {

@@ -3,7 +3,7 @@ kinds of layer: state-space mixers (Mamba-2) and layers that run softmax attenti
 same input.
 
     x_1 = .. = x_S = embed[token]
-    per sublayer q (1: mixer, 2: feed-forward) of a layer, with its own ``in`` [S], ``mix`` [S, S], ``out`` [S]:
+    per sublayer, with its own ``in`` [S], ``mix`` [S, S], ``out`` [S] (hc1 for a layer's mixer, hc2 for its feed-forward):
         y   = sublayer(N(sum_s in[s] x_s; norm_q))
         x_t = sum_s mix[s, t] x_s + out[t] y          (all t from the old streams)
     logits = head N(sum_s x_s; final.norm)            N(z; w) = w z / rms(z)

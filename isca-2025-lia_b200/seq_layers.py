@@ -648,7 +648,7 @@ class GatedRecurrentMixer:
 
 
 class ParallelMixer:
-    """Two mixers on one input, side by side: half the sum of their outputs, each first RMS-normed with a plain weight.  ``left`` is built with
+    """Two mixers fed with one input; what leaves is the mean of the two results, taken after an RMS norm of its own on each.  ``left`` is built with
     the projections of ``right`` riding along on its own (one GEMM for both) if ``shared_projection``.  The call returns the two
     outputs; ``branch_norms`` and ``branch_scale`` say how the residual update that follows joins them (``ops.streams_update``)."""
 
@@ -670,7 +670,7 @@ class ParallelMixer:
 class StateSpaceMixer:
     """Mamba-2's mixer (state-space duality): Win h = z | x | B | C | dt; x, B and C pass a short causal convolution with a bias per channel and
     SiLU; dt = softplus(dt + dt_bias); per head S = exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x (csrc/linear_scan.cu; the heads share
-    B and C in ``groups``); y * silu(z) RMS-normed in ``norm_groups`` equal parts with a plain weight, then Wo.  Step sizes, decays, state and
+    B and C in ``groups``); N(y * silu(z)), the norm's mean taken over each of ``norm_groups`` stretches of the heads, then Wo.  Step sizes, decays, state and
     sums are fp32."""
 
     def __init__(self, w, heads, vdim, state, groups, norm_groups, taps, norm_eps, dtype, device):
